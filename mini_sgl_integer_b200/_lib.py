@@ -1,4 +1,5 @@
-"""ctypes binding of ``libb200int.so`` (the C ABI declared in ``include/b200int.h``).
+"""ctypes binding of the C-ABI libraries: ``libb200int.so`` (``include/b200int.h``, the integer path) and
+``libb200float.so`` (``include/b200float.h``, floating-point models).
 
 There is no fallback: if the library has not been built, or an entry point
 rejects its arguments, the call raises.
@@ -7,14 +8,15 @@ from __future__ import annotations
 
 import ctypes
 import os
-from ctypes import c_char_p, c_int, c_int64, c_void_p
+from ctypes import c_char_p, c_float, c_int, c_int64, c_void_p
 
 import torch
 
 _PKG = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_PKG, "libb200int.so")
+FLOAT_LIB_PATH = os.path.join(_PKG, "libb200float.so")
 
-P, I, L = c_void_p, c_int, c_int64
+P, I, L, F = c_void_p, c_int, c_int64, c_float
 
 # name -> argument types (every function returns int unless listed in _RESTYPES)
 SIGNATURES: dict[str, list] = {
@@ -73,35 +75,60 @@ SIGNATURES: dict[str, list] = {
     "b200_tp_status": [P, I],
     "b200_tp_set_timeout_us": [L],
 }
+FLOAT_SIGNATURES: dict[str, list] = {
+    "b200f_gemm_splits": [L, L, L, L, I],
+    "b200f_gemm": [P, P, P, I, I, L, L, L, L, L, L, L, L, L, L, I, L, I, F, F, P],
+    "b200f_gemm_status": [P, I],
+    "b200f_embed_bigram": [P, P, P, P, P, P, P, P, P, P, I, L, I, L, L, L, L, L, P],
+    "b200f_sublayer_end": [P, I, L, P, P, P, P, P, I, L, P, P, P, I, L, I, L, F, P],
+    "b200f_xielu": [P, I, L, P, I, L, I, L, F, F, P],
+    "b200f_mingru": [P, I, L, P, P, P, P, P, P, P, I, L, I, I, L, P],
+    "b200f_latent_prepare": [P, I, L, L, P, P, P, I, I, P, F, P, P, P, I, L, I, I, I, I, I, I, I, L, P],
+    "b200f_latent_attn_ws_floats": [L, I, I, I],
+    "b200f_latent_attn_splits": [L, I, I, I, I, I, I, I, I],
+    "b200f_latent_attn": [P, P, P, L, P, P, P, P, I, L, I, I, I, I, I, I, I, I, F, I, P, I, P],
+    "b200f_argmax": [P, L, L, L, P, P],
+}
+_SHARED = ("b200_last_error_string", "b200_decode_prepare")      # in every library
 _RESTYPES = {"b200_last_error_string": c_char_p, "b200_attn_workspace_bytes": ctypes.c_size_t,
-             "b200_tp_block_bytes": ctypes.c_size_t}
+             "b200_tp_block_bytes": ctypes.c_size_t, "b200f_latent_attn_ws_floats": ctypes.c_size_t}
 
-_lib = None
+_libs: dict[str, ctypes.CDLL] = {}
 
 
 class B200Error(RuntimeError):
-    """An entry point of libb200int.so returned a negative status."""
+    """An entry point of a library returned a negative status."""
 
     def __init__(self, name: str, code: int, message: str):
         super().__init__(f"{name} failed with status {code}: {message}")
         self.code = code
 
 
-def load() -> ctypes.CDLL:
-    global _lib
-    if _lib is None:
-        if not os.path.exists(LIB_PATH):
+def load(which: str = "int") -> ctypes.CDLL:
+    if which not in _libs:
+        path, signatures = (LIB_PATH, SIGNATURES) if which == "int" else \
+            (FLOAT_LIB_PATH, {**FLOAT_SIGNATURES, **{n: SIGNATURES[n] for n in _SHARED}})
+        if not os.path.exists(path):
             raise RuntimeError(
-                f"{LIB_PATH} is missing: build it with `python -m mini_sgl_integer_b200.build` "
+                f"{path} is missing: build it with `python -m mini_sgl_integer_b200.build` "
                 "(there is no CPU or PyTorch fallback for these kernels)"
             )
-        lib = ctypes.CDLL(LIB_PATH)
-        for name, args in SIGNATURES.items():
+        lib = ctypes.CDLL(path)
+        for name, args in signatures.items():
             fn = getattr(lib, name)  # AttributeError here = header and library disagree
             fn.argtypes = args
             fn.restype = _RESTYPES.get(name, c_int)
-        _lib = lib
-    return _lib
+        _libs[which] = lib
+    return _libs[which]
+
+
+def library_of(name: str) -> ctypes.CDLL:
+    """The library that holds an entry point; one that every library holds comes from a library already in use."""
+    if name in FLOAT_SIGNATURES:
+        return load("float")
+    if name in _SHARED and "int" not in _libs and "float" in _libs:
+        return _libs["float"]
+    return load("int")
 
 
 CALLS = 0      # entry-point calls made through `call` (bench.py counts the launches of a captured step with it)
@@ -109,12 +136,17 @@ CALLS = 0      # entry-point calls made through `call` (bench.py counts the laun
 
 def call(name: str, *args) -> None:
     global CALLS
-    lib = load()
+    lib = library_of(name)
     CALLS += 1
     rc = getattr(lib, name)(*args)
     if rc != 0:
         msg = lib.b200_last_error_string().decode("utf-8", "replace")
         raise B200Error(name, rc, msg)
+
+
+def query(name: str, *args) -> int:
+    """An entry point that returns a number instead of a status."""
+    return getattr(library_of(name), name)(*args)
 
 
 def ptr(t: torch.Tensor | None):

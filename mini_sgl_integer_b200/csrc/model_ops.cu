@@ -1,8 +1,7 @@
-// The two ends of the integer model and the per-step bookkeeping of a decode batch:
+// The two ends of the integer model:
 //   * embedding rows (bf16 table) gathered by token id and converted to Q15.16,
-//   * arg-max over int32 logits rows (lowest index wins ties),
-//   * advancing a decode batch by one token on the device (positions, KV locations, lengths).
-// All three are memory-bound row kernels: 16-byte loads and stores, one CTA (or warp) per row.
+//   * arg-max over int32 logits rows (lowest index wins ties).
+// Both are memory-bound row kernels: 16-byte loads and stores, one CTA (or warp) per row.
 #include <cuda_bf16.h>
 
 #include "common.cuh"
@@ -102,27 +101,6 @@ argmax_rows_kernel(const int32_t* __restrict__ logits, int64_t pitch, int64_t n,
 }
 
 // ---------------------------------------------------------------------------------------------------
-// One decode step of bookkeeping for `batch` sequences, all on the device so that the step can be
-// replayed from a CUDA graph: the new token of sequence b sits at position seq_lens[b]; its KV slot
-// is page_table[b][pos / 16] * 16 + pos % 16; the sequence then has pos + 1 keys.
-// ---------------------------------------------------------------------------------------------------
-__global__ void decode_prepare_kernel(const int32_t* __restrict__ page_table, int64_t pitch, int32_t* __restrict__ seq_lens,
-                                      int32_t* __restrict__ positions, int32_t* __restrict__ out_loc,
-                                      int32_t* __restrict__ kv_lens, int batch, int max_len) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int b = blockIdx.x * blockDim.x + threadIdx.x;
-  if (b >= batch) return;
-  int pos = seq_lens[b];
-  pos = pos < 0 ? 0 : (pos > max_len - 1 ? max_len - 1 : pos);      // a full sequence rewrites its last slot
-  const int page = page_table[(int64_t)b * pitch + (pos >> 4)];
-  positions[b] = pos;
-  out_loc[b] = page * 16 + (pos & 15);
-  kv_lens[b] = pos + 1;
-  seq_lens[b] = pos + 1;
-}
-
-// ---------------------------------------------------------------------------------------------------
 // Per-tensor int8 quantisation of a bf16 tensor with a (multiplier, shift) scale: the quantiser the
 // reference's prefill path applies to q, k and v (quantize_per_tensor_int8_ms).  Two passes: the
 // absolute maximum (bf16 bit patterns of non-negative values order like integers), then the codes.
@@ -193,17 +171,6 @@ extern "C" int b200_argmax_i32(const int32_t* logits, int64_t rows, int64_t n, i
   B200_REQUIRE(rows < (1ll << 31), B200_E_SHAPE, "argmax: too many rows");
   launch_pdl(argmax_rows_kernel, dim3((unsigned)rows), dim3(kArgmaxThreads), 0, (cudaStream_t)s, logits, pitch, n, index_offset, out_idx, out_val);
   return check_launch("argmax_i32");
-}
-
-extern "C" int b200_decode_prepare(const int32_t* page_table, int64_t table_pitch, int32_t* seq_lens, int32_t* positions,
-                                   int32_t* out_loc, int32_t* kv_lens, int batch, int max_len, b200_stream_t s) {
-  B200_REQUIRE(batch >= 0 && max_len > 0 && table_pitch >= (max_len + 15) / 16, B200_E_SHAPE,
-               "decode_prepare: batch=%d max_len=%d table_pitch=%lld", batch, max_len, (long long)table_pitch);
-  if (batch == 0) return B200_OK;
-  B200_REQUIRE(page_table && seq_lens && positions && out_loc && kv_lens, B200_E_NULL, "decode_prepare: null pointer");
-  launch_pdl(decode_prepare_kernel, dim3((batch + 127) / 128), dim3(128), 0, (cudaStream_t)s, page_table, table_pitch, seq_lens, positions, out_loc,
-             kv_lens, batch, max_len);
-  return check_launch("decode_prepare");
 }
 
 extern "C" int b200_quantize_per_tensor_int8_ms(const uint16_t* x_bf16, int64_t n, int8_t* codes, int32_t* mul_shift,
