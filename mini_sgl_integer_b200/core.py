@@ -38,6 +38,8 @@ class Batch:
     out_loc: torch.Tensor = field(init=False, default=None)
     padded_reqs: List[Any] = field(init=False, default=None)
     attn_metadata: Any = field(init=False, default=None)
+    # token rows whose logits are asked for (int64); None: the last token of every request
+    logit_rows: Optional[torch.Tensor] = field(init=False, default=None)
 
     def __post_init__(self) -> None:
         if self.padded_reqs is None:

@@ -61,6 +61,9 @@ class ParallelLMHead(BaseOP):
 
     def _last_tokens(self, x_q15: torch.Tensor) -> torch.Tensor:
         batch = get_global_ctx().batch
+        wanted = getattr(batch, "logit_rows", None)
+        if wanted is not None:
+            return x_q15.index_select(0, wanted)
         if batch.is_prefill:
             idx = batch.attn_metadata.get_last_indices(batch.size)
             x_q15 = x_q15.index_select(0, idx.to(torch.int64))
