@@ -43,6 +43,8 @@ class SefevikLayer(BaseOP):
         if self.mlp is not None:
             self.norm2 = take_f32(state_dict, prefix + "norm2", (self._hidden,), self._device)
             self.mlp.load_state_dict(state_dict, prefix=prefix + "mlp.")
+        else:
+            state_dict.pop(prefix + "norm2", None)         # a gain without a sublayer has nothing to act on
         self.dwa = take_f32(state_dict, prefix + "dwa", (self._id + 2,), self._device)
 
     def forward(self, x_in: torch.Tensor, x: Optional[torch.Tensor], x_mid: torch.Tensor, xt: torch.Tensor, hist: torch.Tensor, md, cache,
