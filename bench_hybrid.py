@@ -228,14 +228,21 @@ def kernel_table(s: dict, q: dict, B: int, prompts: int, n: int, ctx: int) -> di
             lbest = max((lbytes or 0) / pk["hbm_gbs"] / 1e6, (lflops or 0) / pk["int8_tops"] / 1e9)
             out[name]["like"] = {"name": lname, "us": lms * 1e3, "frac": lbest / lms}
 
-    def rotating(make, fn, bytes_each, reps=40):
+    def device_ms(fn, calls=16, reps=5):
+        """Per call, from a captured graph of `calls` calls: small kernels would otherwise be timed at the host's launch rate."""
+        def many():
+            for _ in range(calls):
+                fn()
+        return timed(captured(many, 1).replay, reps) / calls
+
+    def rotating(make, fn, bytes_each):
         copies = [make() for _ in range(max(1, min(16, int(3e8 // max(bytes_each, 1)) + 1)))]
         k = [0]
 
         def run():
             k[0] = (k[0] + 1) % len(copies)
             fn(copies[k[0]])
-        return timed(run, reps)
+        return device_ms(run)
 
     # linears, and the int8 linear of the same (M, N, K)
     from mini_sgl_integer_b200.layers.w8a8_int8 import int8_gemm_q15
@@ -289,20 +296,20 @@ def kernel_table(s: dict, q: dict, B: int, prompts: int, n: int, ctx: int) -> di
     def like_decode():
         rot[0] = (rot[0] + 1) % 4
         decode_attention_int8_paged(q8, qm, qs, pool, rot[0], table, lens, max_len)
-    lms = timed(like_decode, 40)
+    lms = device_ms(like_decode)
     entry("latent attention, decode", ms, 2.0 * B * seen * lat + 2.0 * B * H * (lat + s["rank"]), 2.0 * B * seen * H * (lat + s["rank"]),
           ("attn_decode (int8)", lms, float(B * ctx * q["kv"] * 266), 4.0 * B * ctx * q["heads"] * 128))
     pos, loc, seq, start, plens = prompt_meta(prompts, n, table)
     ql2, o2 = rnd(T, H, lat), torch.empty(T, H, s["rank"], dtype=bf, device="cuda")
     c = rnd(pages, 16, lat)
     tb = table[:prompts].contiguous()
-    ms = timed(lambda: fo.latent_attention(ql2, c, tb, plens, start, sink, o2, s["rank"], s["rot"], s["window"], 0.1, n, n), 10)
+    ms = device_ms(lambda: fo.latent_attention(ql2, c, tb, plens, start, sink, o2, s["rank"], s["rot"], s["window"], 0.1, n, n))
     w = min(n, s["window"])
     pairs = prompts * (w * (w + 1) / 2 + (n - w) * w)
     q8p = torch.randint(-127, 128, (T, q["heads"], 128), dtype=torch.int8, device="cuda")
     qmp = torch.randint(2 ** 30, 2 ** 31, (T, q["heads"]), dtype=torch.int64, device="cuda").to(torch.int32)
     qsp = torch.full((T, q["heads"]), 44, dtype=torch.int32, device="cuda")
-    lms = timed(lambda: prefill_attention_int8_paged(q8p, qmp, qsp, pool, 0, tb, plens, plens, n, n), 10)
+    lms = device_ms(lambda: prefill_attention_int8_paged(q8p, qmp, qsp, pool, 0, tb, plens, plens, n, n))
     entry("latent attention, prompts", ms, 2.0 * T * lat + 2.0 * T * H * (lat + s["rank"]), 2.0 * pairs * H * (lat + s["rank"]),
           ("attn_prefill (int8)", lms, None, 4.0 * prompts * n * (n + 1) / 2 * q["heads"] * 128))
     del pool, q8p, qmp, qsp, ql2, o2, c
@@ -315,26 +322,26 @@ def kernel_table(s: dict, q: dict, B: int, prompts: int, n: int, ctx: int) -> di
         xo, xt = torch.empty_like(x), fo.rows(M, W, bf, "cuda")
         planes = s["depth"] // 2
         xi, ri, wi = (torch.randint(-2 ** 18, 2 ** 18, sh, dtype=torch.int32, device="cuda") for sh in ((M, W), (M, W), (W,)))
-        lms = timed(lambda: fp.fused_add_rmsnorm_quant(xi, ri, wi), 40)
+        lms = device_ms(lambda: fp.fused_add_rmsnorm_quant(xi, ri, wi))
         like = ("add + RMSNorm + quant rows (int)", lms, 13.0 * M * W, None)
-        entry(f"sublayer end M={M}", timed(lambda: fo.sublayer_end(y, x, nw, 1e-6, xo, xt, bf), 40), 14.0 * M * W, None, like)
+        entry(f"sublayer end M={M}", device_ms(lambda: fo.sublayer_end(y, x, nw, 1e-6, xo, xt, bf)), 14.0 * M * W, None, like)
         h, coef = torch.randn(planes + 1, M, W, device="cuda"), torch.randn(planes + 1, device="cuda")
         entry(f"sublayer end + depth average over {planes + 1} M={M}",
-              timed(lambda: fo.sublayer_end(y, x, nw, 1e-6, xo, xt, bf, hist=h, planes=planes, coef=coef, hist_out=h[planes]), 40),
+              device_ms(lambda: fo.sublayer_end(y, x, nw, 1e-6, xo, xt, bf, hist=h, planes=planes, coef=coef, hist_out=h[planes])),
               (18.0 + 4.0 * planes) * M * W, None, like)
         del h, y, x, xo, xt, xi, ri
         gru = s["gru"]
         zug, bz = torch.randn(1, M, 3 * gru, device="cuda"), torch.randn(gru, device="cuda")
         state, yo = torch.zeros(max(B, prompts), gru, device="cuda"), fo.rows(M, gru, bf, "cuda")
         gu = torch.randint(-2 ** 18, 2 ** 18, (M, 2 * (gru - gru % 128)), dtype=torch.int32, device="cuda")
-        lms = timed(lambda: fp.silu_mul_fwht_quant(gu, 128), 40)
+        lms = device_ms(lambda: fp.silu_mul_fwht_quant(gu, 128))
         like = ("SiLU * up + rotation + quant rows (int)", lms, 9.0 * M * (gru - gru % 128), None)
         if M == B:
             sl, p1 = torch.arange(B, dtype=torch.int32, device="cuda"), torch.ones(B, dtype=torch.int32, device="cuda")
-            entry(f"minGRU step M={M}", timed(lambda: fo.mingru(zug, bz, bz, state, sl, p1, None, B, yo), 40), 22.0 * M * gru, None, like)
+            entry(f"minGRU step M={M}", device_ms(lambda: fo.mingru(zug, bz, bz, state, sl, p1, None, B, yo)), 22.0 * M * gru, None, like)
         else:
             sl = torch.arange(prompts, dtype=torch.int32, device="cuda")
-            entry(f"minGRU scan M={M}", timed(lambda: fo.mingru(zug, bz, bz, state, sl, pos, start, prompts, yo), 20), 14.0 * M * gru, None, like)
+            entry(f"minGRU scan M={M}", device_ms(lambda: fo.mingru(zug, bz, bz, state, sl, pos, start, prompts, yo)), 14.0 * M * gru, None, like)
         del zug, gu, yo
         nq = H * (s["dim"] + s["rot"]) + lat
         qd, cache = torch.randn(1, M, nq, device="cuda"), torch.zeros(pages, 16, lat, dtype=bf, device="cuda")
@@ -348,10 +355,10 @@ def kernel_table(s: dict, q: dict, B: int, prompts: int, n: int, ctx: int) -> di
         qkv = torch.randint(-2 ** 18, 2 ** 18, (M, (q["heads"] + 2 * q["kv"]) * 128), dtype=torch.int32, device="cuda")
         cs = rope_cache_q15(16).cuda()
         nwq = torch.randint(2 ** 11, 2 ** 13, (128,), dtype=torch.int32, device="cuda")
-        lms = timed(lambda: qkv_rope_quant_store(pp, qkv, q["heads"], pool, 0, ll, cs, nwq, nwq), 40)
+        lms = device_ms(lambda: qkv_rope_quant_store(pp, qkv, q["heads"], pool, 0, ll, cs, nwq, nwq))
         lb = M * ((q["heads"] + 2 * q["kv"]) * 512.0 + q["heads"] * 136.0 + q["kv"] * 266.0)
         dn = torch.ones(s["rank"], device="cuda")
-        ms = timed(lambda: fo.latent_prepare(qd, pp, ll, rope, dn, 1e-6, qn, qq, cache, H, s["dim"], s["rot"], s["rank"]), 40)
+        ms = device_ms(lambda: fo.latent_prepare(qd, pp, ll, rope, dn, 1e-6, qn, qq, cache, H, s["dim"], s["rot"], s["rank"]))
         entry(f"latent prepare M={M}", ms, M * (4.0 * nq + 2.0 * H * (s["dim"] + s["rot"]) + 2.0 * lat), None, ("qkv_prepare rows (int)", lms, lb, None))
         del qd, cache, qn, qq, pool, qkv
         torch.cuda.empty_cache()

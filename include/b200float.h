@@ -93,6 +93,8 @@ B200_API int b200f_latent_attn(const void* q_lat, const void* cache, const int32
                                int out_pitch, int window, float scale, int key_splits, float* ws, int simple,
                                b200_stream_t s);
 
+B200_API int b200f_latent_attn_status(int* out_host, int reset);   /* as b200f_gemm_status: 5 copying warp, 6 consumer */
+
 /* ---- Row-wise arg-max of fp32 logits, the lowest index wins ties. */
 B200_API int b200f_argmax(const float* logits, int64_t rows, int64_t n, int64_t pitch, int32_t* out_idx, b200_stream_t s);
 

@@ -87,6 +87,7 @@ FLOAT_SIGNATURES: dict[str, list] = {
     "b200f_latent_attn_ws_floats": [L, I, I, I],
     "b200f_latent_attn_splits": [L, I, I, I, I, I, I, I, I],
     "b200f_latent_attn": [P, P, P, L, P, P, P, P, I, L, I, I, I, I, I, I, I, I, F, I, P, I, P],
+    "b200f_latent_attn_status": [P, I],
     "b200f_argmax": [P, L, L, L, P, P],
 }
 _SHARED = ("b200_last_error_string", "b200_decode_prepare")      # in every library

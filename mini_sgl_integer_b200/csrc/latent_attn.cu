@@ -4,14 +4,17 @@
 //                         the latent, cache store; one CTA per token.
 // latent_attn_mma_kernel  bf16, prompts and decode alike.  Queries live in the latent space (the caller multiplied them by
 //                         the key up-projection), so every head sees the same keys and a query tile is
-//                         (tokens x heads) rows: 16 rows for a decode step with few heads, 64 rows for prompts.  Key tiles
-//                         are gathered from the pages with cp.async into a double buffer; a tile serves the scores (all
-//                         kv_rank + rot_dim columns) and the values (its first kv_rank columns).  Eight warps: the scores are
-//                         split over (row groups x key groups), the output over (row groups x column groups), with the
-//                         probabilities exchanged through shared memory.  Scores, softmax and accumulators are fp32.
-//                         Long key ranges of small batches are split over CTAs and merged by latent_merge_kernel.
+//                         (tokens x heads) rows: 16 or 32 rows for a decode step, 64 rows for prompts.  A warp gathers
+//                         key tiles from the pages with bulk copies (one key row per lane) into an mbarrier ring; a tile
+//                         serves the scores (all kv_rank + rot_dim columns) and the values (its first kv_rank columns).
+//                         The other warps form row groups of 16 rows; inside a group they split the reduction of the
+//                         scores (each keeps its slice of the queries in registers), then the rows of the softmax, then
+//                         the columns of the output, and meet at two named barriers per tile.  Scores, softmax and
+//                         accumulators are fp32.  Long key ranges of small batches are split over CTAs and merged by
+//                         latent_merge_kernel.
 // latent_attn_kernel      any size, any type, one CTA per (token, head); the 32-bit path.
 #include "float_common.cuh"
+#include "umma.cuh"
 
 namespace b200 {
 
@@ -169,18 +172,8 @@ latent_attn_kernel(const AttnParams p, const T* __restrict__ q_lat, const T* __r
 }
 
 // ---------------------------------------------------------------------------------------------------
-__device__ __forceinline__ unsigned sm_addr(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void cp_async16(unsigned dst, const void* src, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void ldsm_x4(unsigned (&r)[4], unsigned addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x2(unsigned& r0, unsigned& r1, unsigned addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
 __device__ __forceinline__ void ldsm_x4_t(unsigned (&r)[4], unsigned addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -191,34 +184,66 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const unsigned (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// MT row groups of 16 query rows, NK keys per tile, up to NC16 16-column pieces of the output per warp.
-template <int MT, int NK>
+// MT row groups of 16 query rows, WARPS warps that compute, a ring of STAGES tiles of 32 keys; a warp's
+// slice of the reduction has up to KS steps of 16, its slice of the output up to NC pieces of 16 columns.
+constexpr int kKeyTile = 32;
+constexpr int kScorePitch = kKeyTile + 8;      // values per staged row (fp32 scores, bf16 weights): conflict-free both ways
+
+template <int MT, int WARPS, int STAGES>
 struct AttnShape {
-  static constexpr int kRows = 16 * MT, kGroups = 8 / MT, kKeysPerWarp = NK / kGroups;
-  static constexpr int kPPitch = NK + 8;                                     // bf16, conflict-free for ldmatrix
+  static constexpr int kRows = 16 * MT, kGroup = WARPS / MT;
+  static constexpr bool kCopyWarp = WARPS == 4;
+  static constexpr int kThreads = 32 * (WARPS + (kCopyWarp ? 1 : 0));
   static size_t smem(int d16) {
-    return (size_t)(kRows + 2 * NK) * (d16 + 8) * 2 + (size_t)kRows * kPPitch * 2 + (size_t)2 * kRows * kGroups * 4;
+    return (size_t)STAGES * kKeyTile * (d16 + 8) * 2 + (size_t)kGroup * kRows * kScorePitch * 4 + (size_t)kRows * kScorePitch * 2 +
+           (size_t)3 * kRows * 4 + 2 * STAGES * 8;
   }
 };
 
-template <int MT, int NK, int NC16>
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ float exp2_approx(float v) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+__device__ __forceinline__ void bulk_load(unsigned dst, const void* src, unsigned bytes, unsigned bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+__device__ __forceinline__ void group_sync(int group, int threads) {
+  asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "r"(threads) : "memory");
+}
+
+template <int MT, int WARPS, int STAGES, int KS, int NC, int MINB>
+__global__ void __launch_bounds__((AttnShape<MT, WARPS, STAGES>::kThreads), MINB)
 latent_attn_mma_kernel(const AttnParams p, const bf16* __restrict__ q_lat, const bf16* __restrict__ cache, bf16* __restrict__ out) {
-  using S = AttnShape<MT, NK>;
-  constexpr int R = S::kRows, G = S::kGroups, KW = S::kKeysPerWarp, KT = KW / 8;
-  static_assert(KW >= 8 && KW % 8 == 0, "key tile too small for this many warps");
+  using S = AttnShape<MT, WARPS, STAGES>;
+  constexpr int R = S::kRows, G = S::kGroup, NK = kKeyTile, RW = 16 / G, U = RW / 4;   // RW: softmax rows per warp
+  constexpr bool kCopyWarp = S::kCopyWarp;
+  static_assert(G * MT == WARPS && RW % 4 == 0 && (kCopyWarp || STAGES > 2), "shape");
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int D = p.kv_rank + p.rot_dim;
   const int d16 = (D + 15) & ~15, ld = d16 + 8;
-  bf16* qs = reinterpret_cast<bf16*>(smem_raw);                              // [R][ld]
-  bf16* ks = qs + R * ld;                                                    // [2][NK][ld]
-  bf16* ps = ks + 2 * NK * ld;                                               // [R][kPPitch]
-  float* red = reinterpret_cast<float*>(ps + R * S::kPPitch);                // [R][G] maxima; sums behind them at the end
+  bf16* ks = reinterpret_cast<bf16*>(smem_raw);                              // [STAGES][NK][ld]
+  float* sp = reinterpret_cast<float*>(ks + STAGES * NK * ld);               // [G][R][kScorePitch] partial scores
+  bf16* ps = reinterpret_cast<bf16*>(sp + G * R * kScorePitch);              // [R][kScorePitch] weights
+  float* row_alpha = reinterpret_cast<float*>(ps + R * kScorePitch);         // [R], then [R][2] maximum and sum
+  float* row_ml = row_alpha + R;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(row_ml + 2 * R);              // full[STAGES], empty[STAGES]
 
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int rg = warp / G, kg = warp % G;
+  const unsigned full0 = smem_u32(bars), empty0 = smem_u32(bars + STAGES);
   const int split = blockIdx.x % p.splits, q_tile = blockIdx.x / p.splits, hg = blockIdx.y, seq = blockIdx.z;
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < STAGES; ++s) {
+      mbar_init(full0 + 8 * s, 1);
+      mbar_init(empty0 + 8 * s, WARPS);
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  for (int r = warp; r < STAGES * NK; r += S::kThreads / 32)                        // columns behind a row's copied part stay zero
+    for (int c = p.lat_pitch + lane; c < d16; c += 32) ks[r * ld + c] = __float2bfloat16_rn(0.0f);
+  __syncthreads();
   pdl_wait();
   const int start = p.seq_start ? p.seq_start[seq] : seq;
   const int count = p.seq_start ? p.seq_start[seq + 1] - start : 1;
@@ -231,192 +256,207 @@ latent_attn_mma_kernel(const AttnParams p, const bf16* __restrict__ q_lat, const
   const int key_lo = first_key(pos0, p.window), key_hi = pos0 + ntok;        // keys [key_lo, key_hi)
   const int all_tiles = (key_hi - key_lo + NK - 1) / NK, per = (all_tiles + p.splits - 1) / p.splits;
   const int tile0 = split * per, tile1 = min(all_tiles, tile0 + per);
+
+  // Copies, one key row per lane and tile; rows behind the last key repeat it (they are masked).  A tile's cache row is
+  // looked up one tile ahead.  Small CTAs have a warp for this; the large ones, whose registers an extra warp would cut,
+  // let warp 0 do it two tiles before the ring is full again.
   const int32_t* pages = p.page_table + (int64_t)seq * p.table_pitch;
-  const int chunks = p.lat_pitch / 8;                                        // 16-byte pieces of a row; the rest stays zero
-
-  // query rows, and zeros behind the rows' ends (query and key tiles)
-  for (int r = warp; r < R; r += 8) {
-    const int tok = r / nh, hd = r - tok * nh;
-    const bf16* src = q_lat + ((int64_t)(start + tok0 + (r < rows ? tok : 0)) * p.heads + h0 + (r < rows ? hd : 0)) * p.lat_pitch;
-    for (int c = lane; c < chunks; c += 32) cp_async16(sm_addr(qs + r * ld + 8 * c), src + 8 * c, r < rows);
-    for (int c = chunks * 8 + lane; c < d16; c += 32) qs[r * ld + c] = __float2bfloat16_rn(0.0f);
-  }
-  for (int r = warp; r < 2 * NK; r += 8)
-    for (int c = chunks * 8 + lane; c < d16; c += 32) ks[r * ld + c] = __float2bfloat16_rn(0.0f);
-
-  auto load_tile = [&](int tile, int buf) {
-    const int k0 = key_lo + tile * NK;
-    int page[NK / 8];
-#pragma unroll
-    for (int i = 0; i < NK / 8; ++i) {
-      const int key = k0 + warp + 8 * i;
-      page[i] = key < key_hi ? __ldg(pages + key / kPage) : -1;
-    }
-#pragma unroll
-    for (int i = 0; i < NK / 8; ++i) {
-      const int r = warp + 8 * i, key = k0 + r;
-      const bool ok = page[i] >= 0;
-      const bf16* src = cache + ((int64_t)(ok ? page[i] : 0) * kPage + key % kPage) * p.lat_pitch;
-      const unsigned dst = sm_addr(ks + (buf * NK + r) * ld);
-      for (int c = lane; c < chunks; c += 32) cp_async16(dst + 16 * c, src + 8 * c, ok);
+  const unsigned bytes = (unsigned)p.lat_pitch * 2;
+  int64_t src_row = 0;
+  auto look_up = [&](int tile) {
+    if (tile < tile1) {
+      const int key = min(key_lo + tile * NK + lane, key_hi - 1);
+      src_row = (int64_t)__ldg(pages + key / kPage) * kPage + key % kPage;
     }
   };
-  if (tile0 < tile1) load_tile(tile0, 0);
-  cp_async_commit();
-
-  // this lane's two accumulator rows and the keys they may see
-  int vis_lo[2], vis_hi[2];
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = rg * 16 + (lane >> 2) + 8 * i;
-    const int pos = pos0 + r / nh;
-    vis_hi[i] = r < rows ? pos : -1;
-    vis_lo[i] = p.window > 0 ? pos - p.window + 1 : 0;
+  auto copy_tile = [&](int tile) {               // needs look_up(tile); all lanes of one warp; false after an expired wait
+    const unsigned i = tile - tile0, s = i % STAGES;
+    const int64_t row = src_row;
+    look_up(tile + 1);
+    if (!__all_sync(FULL_MASK, mbar_wait(empty0 + 8 * s, ((i / STAGES) & 1) ^ 1, 5))) return false;
+    if (lane == 0) mbar_expect_tx(full0 + 8 * s, bytes * NK);
+    __syncwarp();
+    bulk_load(smem_u32(ks + (s * NK + lane) * ld), cache + row * p.lat_pitch, bytes, full0 + 8 * s);
+    return true;
+  };
+  bool ok = true;
+  if (kCopyWarp) {
+    if (warp == WARPS) {
+      look_up(tile0);
+      for (int tile = tile0; tile < tile1 && ok; ++tile) ok = copy_tile(tile);
+      return;
+    }
+  } else if (warp == 0) {
+    look_up(tile0);
+    for (int tile = tile0; tile < min(tile1, tile0 + STAGES - 2) && ok; ++tile) ok = copy_tile(tile);
   }
-  float acc[NC16][2][4];
+
+  const int rg = warp / G, kg = warp % G;
+  // this warp's slice of the reduction and its query fragments (row-major A fragments straight from global memory)
+  const int k16 = d16 / 16, k_per = (k16 + G - 1) / G, k_lo = kg * k_per, k_n = max(0, min(k_per, k16 - k_lo));
+  unsigned qf[KS][4];
+  {
+    const bf16* src[2];
+    bool live[2];
 #pragma unroll
-  for (int i = 0; i < NC16; ++i)
+    for (int i = 0; i < 2; ++i) {
+      const int r = rg * 16 + (lane >> 2) + 8 * i, tok = r / nh;
+      live[i] = r < rows;
+      src[i] = q_lat + ((int64_t)(start + tok0 + (live[i] ? tok : 0)) * p.heads + h0 + (live[i] ? r - tok * nh : 0)) * p.lat_pitch;
+    }
+#pragma unroll
+    for (int i = 0; i < KS; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int col = (k_lo + i) * 16 + 8 * (j >> 1) + 2 * (lane & 3);
+        qf[i][j] = (i < k_n && live[j & 1] && col < p.lat_pitch) ? __ldg(reinterpret_cast<const unsigned*>(src[j & 1] + col)) : 0u;
+      }
+  }
+  // the rows whose softmax this lane works on (eight lanes per row, four keys each), and the keys they may see
+  int vis_lo[U], vis_hi[U];
+  float m[U], l[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int r = rg * 16 + kg * RW + 4 * u + (lane >> 3), pos = pos0 + r / nh;
+    vis_hi[u] = r < rows ? pos : -1;
+    vis_lo[u] = p.window > 0 ? pos - p.window + 1 : 0;
+    m[u] = -INFINITY;
+    l[u] = 0.0f;
+  }
+  float acc[NC][2][4];
+#pragma unroll
+  for (int i = 0; i < NC; ++i)
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int k = 0; k < 4; ++k) acc[i][j][k] = 0.0f;
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
-  const int c16 = (p.kv_rank + 15) / 16, c_per = (c16 + G - 1) / G;          // 16-column pieces of the output, per column group
+  const int c16 = (p.kv_rank + 15) / 16, c_per = (c16 + G - 1) / G;          // 16-column pieces of the output per warp
   const int c_lo = kg * c_per, c_n = max(0, min(c_per, c16 - c_lo));
+  const unsigned k_lane = ((lane & 7) + ((lane >> 4) << 3)) * ld + k_lo * 16 + ((lane >> 3) & 1) * 8;
+  const unsigned v_lane = (lane & 15) * ld + c_lo * 16 + (lane >> 4) * 8;
+  const int frag = (rg * 16 + (lane >> 2)) * kScorePitch + 2 * (lane & 3);
+  const unsigned pa = smem_u32(ps + (rg * 16 + (lane & 15)) * kScorePitch + (lane >> 4) * 8);
 
   for (int tile = tile0; tile < tile1; ++tile) {
-    const int buf = (tile - tile0) & 1;
-    const bf16* kt = ks + buf * NK * ld;
-    cp_async_wait<0>();
-    __syncthreads();                                                         // tile arrived; the other buffer is free
-    if (tile + 1 < tile1) load_tile(tile + 1, buf ^ 1);
-    cp_async_commit();
-    // scores: 16 rows x KW keys per warp, two accumulator sets to shorten the dependency chain
-    float s[KT][4], s2[KT][4];
+    if (!kCopyWarp && warp == 0 && ok && tile + STAGES - 2 < tile1) ok = copy_tile(tile + STAGES - 2);
+    const unsigned it = tile - tile0, slot = it % STAGES;
+    const bf16* kt = ks + slot * NK * ld;
+    if (ok) ok = mbar_wait(full0 + 8 * slot, (it / STAGES) & 1, 6);
+    __syncwarp();
+    // partial scores: 16 rows x 32 keys over this warp's slice of the reduction
+    float s[NK / 8][4];
 #pragma unroll
-    for (int i = 0; i < KT; ++i)
+    for (int i = 0; i < NK / 8; ++i)
 #pragma unroll
-      for (int k = 0; k < 4; ++k) s[i][k] = s2[i][k] = 0.0f;
-    const unsigned qa = sm_addr(qs + (rg * 16 + (lane & 15)) * ld + (lane >> 4) * 8);
-    const unsigned kb4 = sm_addr(kt + (kg * KW + (lane & 7) + ((lane >> 4) << 3)) * ld + ((lane >> 3) & 1) * 8);
-    const unsigned kb2 = sm_addr(kt + (kg * KW + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
-    auto score_step = [&](int k, float (&dst)[KT][4]) {
-      unsigned a[4];
-      ldsm_x4(a, qa + 2 * k);
-      if (KT == 1) {
-        unsigned b0, b1;
-        ldsm_x2(b0, b1, kb2 + 2 * k);
-        mma_bf16(dst[0], a, b0, b1);
-      } else {
+      for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
+    const unsigned kb = smem_u32(kt + k_lane);
 #pragma unroll
-        for (int i = 0; i + 1 < KT; i += 2) {
+    for (int i = 0; i < KS; ++i) {
+      if (i < k_n) {
+#pragma unroll
+        for (int n = 0; n < NK / 16; ++n) {
           unsigned b[4];
-          ldsm_x4(b, kb4 + (unsigned)(i * 8 * ld * 2) + 2 * k);
-          mma_bf16(dst[i], a, b[0], b[1]);
-          mma_bf16(dst[i + 1 < KT ? i + 1 : i], a, b[2], b[3]);
+          ldsm_x4(b, kb + (unsigned)(n * 16 * ld * 2) + 32 * i);
+          mma_bf16(s[2 * n], qf[i], b[0], b[1]);
+          mma_bf16(s[2 * n + 1], qf[i], b[2], b[3]);
         }
       }
-    };
-    int k = 0;
-#pragma unroll 2
-    for (; k + 16 < d16; k += 32) {
-      score_step(k, s);
-      score_step(k + 16, s2);
     }
-    if (k < d16) score_step(k, s);
-    // mask, scale, row maxima
-    const int key0 = key_lo + tile * NK + kg * KW + 2 * (lane & 3);
-    float mx[2] = {-INFINITY, -INFINITY};
+    float* mine = sp + kg * R * kScorePitch + frag;
 #pragma unroll
-    for (int i = 0; i < KT; ++i)
+    for (int i = 0; i < NK / 8; ++i) {
+      *reinterpret_cast<float2*>(mine + 8 * i) = make_float2(s[i][0], s[i][1]);
+      *reinterpret_cast<float2*>(mine + 8 * kScorePitch + 8 * i) = make_float2(s[i][2], s[i][3]);
+    }
+    group_sync(rg, 32 * G);
+    // softmax step of this warp's rows
+    const int key0 = key_lo + tile * NK + 4 * (lane & 7);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int key = key0 + 8 * i + (j & 1), r = j >> 1;
-        const float v = (key <= vis_hi[r] && key >= vis_lo[r]) ? (s[i][j] + s2[i][j]) * p.scale2 : -INFINITY;
-        s[i][j] = v;
-        mx[r] = fmaxf(mx[r], v);
+    for (int u = 0; u < U; ++u) {
+      const int r = rg * 16 + kg * RW + 4 * u + (lane >> 3);
+      float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+      for (int g = 0; g < G; ++g) {
+        const float4 o = *reinterpret_cast<const float4*>(sp + (g * R + r) * kScorePitch + 4 * (lane & 7));
+        v.x += o.x; v.y += o.y; v.z += o.z; v.w += o.w;
       }
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(FULL_MASK, mx[r], 1));
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(FULL_MASK, mx[r], 2));
-      if ((lane & 3) == 0) red[(rg * 16 + (lane >> 2) + 8 * r) * G + kg] = mx[r];
+      v.x = (key0 <= vis_hi[u] && key0 >= vis_lo[u]) ? v.x * p.scale2 : -INFINITY;
+      v.y = (key0 + 1 <= vis_hi[u] && key0 + 1 >= vis_lo[u]) ? v.y * p.scale2 : -INFINITY;
+      v.z = (key0 + 2 <= vis_hi[u] && key0 + 2 >= vis_lo[u]) ? v.z * p.scale2 : -INFINITY;
+      v.w = (key0 + 3 <= vis_hi[u] && key0 + 3 >= vis_lo[u]) ? v.w * p.scale2 : -INFINITY;
+      float mn = fmaxf(fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w)), m[u]);
+      mn = fmaxf(mn, __shfl_xor_sync(FULL_MASK, mn, 1));
+      mn = fmaxf(mn, __shfl_xor_sync(FULL_MASK, mn, 2));
+      mn = fmaxf(mn, __shfl_xor_sync(FULL_MASK, mn, 4));
+      const float mu = mn == -INFINITY ? 0.0f : mn;                          // no visible key so far: every weight is 0
+      const float alpha = exp2_approx(m[u] - mu);
+      m[u] = mn;
+      v.x = exp2_approx(v.x - mu); v.y = exp2_approx(v.y - mu); v.z = exp2_approx(v.z - mu); v.w = exp2_approx(v.w - mu);
+      l[u] = fmaf(l[u], alpha, (v.x + v.y) + (v.z + v.w));
+      *reinterpret_cast<uint2*>(ps + r * kScorePitch + 4 * (lane & 7)) = make_uint2(f32_to_bf16x2(v.x, v.y), f32_to_bf16x2(v.z, v.w));
+      if ((lane & 7) == 0) row_alpha[r] = alpha;
     }
-    __syncthreads();
-    float alpha[2], mu[2];
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float mn = m[r];
-#pragma unroll
-      for (int g = 0; g < G; ++g) mn = fmaxf(mn, red[(rg * 16 + (lane >> 2) + 8 * r) * G + g]);
-      mu[r] = mn == -INFINITY ? 0.0f : mn;                                   // no visible key so far: every weight is 0
-      alpha[r] = exp2f(m[r] - mu[r]);
-      m[r] = mn;
-      l[r] *= alpha[r];
-    }
-#pragma unroll
-    for (int i = 0; i < KT; ++i) {
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        s[i][j] = exp2f(s[i][j] - mu[j >> 1]);
-        l[j >> 1] += s[i][j];
-      }
-#pragma unroll
-      for (int r = 0; r < 2; ++r)
-        *reinterpret_cast<unsigned*>(ps + (rg * 16 + (lane >> 2) + 8 * r) * S::kPPitch + kg * KW + 8 * i + 2 * (lane & 3)) =
-            f32_to_bf16x2(s[i][2 * r], s[i][2 * r + 1]);
-    }
-    __syncthreads();
+    group_sync(rg, 32 * G);
     // output: 16 rows x this warp's columns
+    const float a0 = row_alpha[rg * 16 + (lane >> 2)], a1 = row_alpha[rg * 16 + (lane >> 2) + 8];
+    if (__any_sync(FULL_MASK, a0 != 1.0f || a1 != 1.0f)) {
 #pragma unroll
-    for (int i = 0; i < NC16; ++i)
+      for (int i = 0; i < NC; ++i)
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        acc[i][j][0] *= alpha[0]; acc[i][j][1] *= alpha[0];
-        acc[i][j][2] *= alpha[1]; acc[i][j][3] *= alpha[1];
-      }
-    const unsigned pa = sm_addr(ps + (rg * 16 + (lane & 15)) * S::kPPitch + (lane >> 4) * 8);
-    const unsigned vb = sm_addr(kt + (lane & 15) * ld + c_lo * 16 + (lane >> 4) * 8);
+        for (int j = 0; j < 2; ++j) {
+          acc[i][j][0] *= a0; acc[i][j][1] *= a0;
+          acc[i][j][2] *= a1; acc[i][j][3] *= a1;
+        }
+    }
+    const unsigned vb = smem_u32(kt + v_lane);
 #pragma unroll
-    for (int kk = 0; kk < NK; kk += 16) {
+    for (int kk = 0; kk < NK / 16; ++kk) {
       unsigned a[4];
-      ldsm_x4(a, pa + 2 * kk);
+      ldsm_x4(a, pa + 32 * kk);
 #pragma unroll
-      for (int i = 0; i < NC16; ++i) {
+      for (int i = 0; i < NC; ++i) {
         if (i < c_n) {
           unsigned b[4];
-          ldsm_x4_t(b, vb + (unsigned)(kk * ld * 2) + 32 * i);
+          ldsm_x4_t(b, vb + (unsigned)(kk * 16 * ld * 2) + 32 * i);
           mma_bf16(acc[i][0], a, b[0], b[1]);
           mma_bf16(acc[i][1], a, b[2], b[3]);
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(empty0 + 8 * slot);
   }
-  cp_async_wait<0>();
-  // row sums over the key groups
-  float* sums = red + R * G;
+  // maxima and sums to the lanes that hold the output
 #pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    l[r] += __shfl_xor_sync(FULL_MASK, l[r], 1);
-    l[r] += __shfl_xor_sync(FULL_MASK, l[r], 2);
-    if ((lane & 3) == 0) sums[(rg * 16 + (lane >> 2) + 8 * r) * G + kg] = l[r];
+  for (int u = 0; u < U; ++u) {
+    l[u] += __shfl_xor_sync(FULL_MASK, l[u], 1);
+    l[u] += __shfl_xor_sync(FULL_MASK, l[u], 2);
+    l[u] += __shfl_xor_sync(FULL_MASK, l[u], 4);
+    if ((lane & 7) == 0) {
+      const int r = rg * 16 + kg * RW + 4 * u + (lane >> 3);
+      row_ml[2 * r] = m[u];
+      row_ml[2 * r + 1] = l[u];
+    }
   }
-  __syncthreads();
+  group_sync(rg, 32 * G);
+  if (!ok) {                                      // a copy did not arrive in time (the status word says so): wait for the
+    for (int t = max(tile0, tile1 - STAGES); t < tile1; ++t)                 // last ones once more and leave
+      mbar_wait(full0 + 8 * ((t - tile0) % STAGES), ((t - tile0) / STAGES) & 1, 6);
+    return;
+  }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = rg * 16 + (lane >> 2) + 8 * r;
     if (row >= rows) continue;
-    float sum = 0.0f;
-#pragma unroll
-    for (int g = 0; g < G; ++g) sum += sums[row * G + g];
+    const float mr = row_ml[2 * row], sum = row_ml[2 * row + 1];
     const int tok = row / nh, hd = h0 + row - tok * nh;
     const int64_t gr = (int64_t)(start + tok0 + tok) * p.heads + hd;
     if (p.splits == 1) {
-      const float sink2 = __ldg(p.sink + hd) * kLog2e, mf = fmaxf(m[r], sink2);
-      const float inv = exp2f(m[r] - mf) / (sum * exp2f(m[r] - mf) + exp2f(sink2 - mf));
+      const float sink2 = __ldg(p.sink + hd) * kLog2e, mf = fmaxf(mr, sink2);
+      const float w = exp2f(mr - mf), inv = w / (sum * w + exp2f(sink2 - mf));
       bf16* dst = out + gr * p.out_pitch;
 #pragma unroll
-      for (int i = 0; i < NC16; ++i)
+      for (int i = 0; i < NC; ++i)
         if (i < c_n) {
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
@@ -431,11 +471,11 @@ latent_attn_mma_kernel(const AttnParams p, const bf16* __restrict__ q_lat, const
       float* dst = p.ws + ((int64_t)split * all + gr) * p.kv_rank;
       if (kg == 0 && (lane & 3) == 0) {
         float* ml = p.ws + (int64_t)p.splits * all * p.kv_rank + ((int64_t)split * all + gr) * 2;
-        ml[0] = m[r];
+        ml[0] = mr;
         ml[1] = sum;
       }
 #pragma unroll
-      for (int i = 0; i < NC16; ++i)
+      for (int i = 0; i < NC; ++i)
         if (i < c_n) {
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
@@ -475,52 +515,42 @@ latent_merge_kernel(const AttnParams p, bf16* __restrict__ out) {
 }
 
 // ----------------------------------------------------------------------------- host side
-struct AttnPlan { int mt, nk, nc16; };      // mt = 0: the plain kernel
+// Kernel variants: row groups, consumer warps, ring slots, limits of a warp's slices, CTAs per SM.  A decode step runs on
+// small CTAs that share an SM; more than 16 heads with a wide latent become several CTAs whose keys meet in L2.
+#define B200_ATTN_VARIANTS(X) \
+  X(1, 4, 4, 5, 4, 2) X(1, 4, 2, 9, 8, 2) X(1, 4, 2, 17, 16, 1) \
+  X(2, 8, 4, 5, 4, 2) \
+  X(4, 8, 4, 5, 4, 1) X(4, 8, 4, 10, 8, 1) X(4, 8, 4, 18, 16, 1)
+
+struct AttnPlan { int mt, warps, stages, ks, nc, minb; };      // mt = 0: the plain kernel
 
 static AttnPlan plan_attn(int max_q, int heads, int kv_rank, int rot_dim) {
-  const int d16 = (kv_rank + rot_dim + 15) & ~15, c16 = (kv_rank + 15) / 16;
-  const size_t limit = 227 * 1024;
+  const int d16 = (kv_rank + rot_dim + 15) & ~15, k16 = d16 / 16, c16 = (kv_rank + 15) / 16;
   const int64_t rows = (int64_t)max_q * heads;
-  const int want = rows <= 16 ? 1 : (rows <= 32 ? 2 : 4);
-  for (int mt = want; mt >= 1; mt >>= 1) {
-    const int per = (c16 * mt + 7) / 8;
-    if (mt == 4 && per <= 16) {
-      const int nc = per <= 4 ? 4 : (per <= 8 ? 8 : 16);
-      if (AttnShape<4, 64>::smem(d16) <= limit) return {4, 64, nc};
-      if (AttnShape<4, 32>::smem(d16) <= limit) return {4, 32, nc};
-    }
-    if (mt == 2 && per <= 8) {
-      const int nc = per <= 4 ? 4 : 8;
-      if (AttnShape<2, 64>::smem(d16) <= limit) return {2, 64, nc};
-      if (AttnShape<2, 32>::smem(d16) <= limit) return {2, 32, nc};
-    }
-    if (mt == 1 && per <= 8 && AttnShape<1, 64>::smem(d16) <= limit) return {1, 64, per <= 4 ? 4 : 8};
+  for (int want = rows <= 16 ? 1 : (rows <= 32 ? 2 : 4); want >= 1; want >>= 1) {
+#define B200_ATTN_FITS(MT_, W_, ST_, KS_, NC_, MB_)                                                              \
+  if (want == MT_ && (k16 + W_ / MT_ - 1) / (W_ / MT_) <= KS_ && (c16 + W_ / MT_ - 1) / (W_ / MT_) <= NC_ &&     \
+      AttnShape<MT_, W_, ST_>::smem(d16) <= 227 * 1024)                                                          \
+    return {MT_, W_, ST_, KS_, NC_, MB_};
+    B200_ATTN_VARIANTS(B200_ATTN_FITS)
+#undef B200_ATTN_FITS
   }
-  return {0, 0, 0};
+  return {0, 0, 0, 0, 0, 0};
 }
 
-static int attn_sm_count() {
-  static int n = 0;
-  if (n == 0) {
-    int dev = 0;
-    if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n <= 0) n = 148;
-  }
-  return n;
-}
-
-template <int MT, int NK, int NC16>
+template <int MT, int WARPS, int STAGES, int KS, int NC, int MINB>
 static int launch_mma(const AttnParams& p, const bf16* q, const bf16* cache, bf16* out, dim3 grid, int d16, cudaStream_t st) {
-  const size_t smem = AttnShape<MT, NK>::smem(d16);
-  cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NK, NC16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = AttnShape<MT, WARPS, STAGES>::smem(d16);
+  cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, WARPS, STAGES, KS, NC, MINB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "latent_attn: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
-  launch_pdl(latent_attn_mma_kernel<MT, NK, NC16>, grid, dim3(256), smem, st, p, q, cache, out);
+  launch_pdl(latent_attn_mma_kernel<MT, WARPS, STAGES, KS, NC, MINB>, grid, dim3(AttnShape<MT, WARPS, STAGES>::kThreads), smem, st, p, q, cache, out);
   return check_launch("latent_attn");
 }
 
-static int tiles_for(int max_q, int max_kv, int window, int tokens_per_cta, int nk) {
+static int tiles_for(int max_q, int max_kv, int window, int tokens_per_cta) {
   int64_t span = max_kv;
   if (window > 0 && span > (int64_t)window + tokens_per_cta - 1) span = (int64_t)window + tokens_per_cta - 1;
-  return (int)((span + nk - 1) / nk);
+  return (int)((span + kKeyTile - 1) / kKeyTile);
 }
 
 }  // namespace b200
@@ -560,8 +590,8 @@ extern "C" int b200f_latent_attn_splits(int64_t tokens, int batch, int max_q, in
   if (pl.mt == 0) return 1;
   const int rows = 16 * pl.mt, hpc = heads < rows ? heads : rows, tpc = rows / hpc;
   const int64_t ctas = (int64_t)((max_q + tpc - 1) / tpc) * ((heads + hpc - 1) / hpc) * batch;
-  const int tiles = tiles_for(max_q, max_kv, window, tpc, pl.nk);
-  int64_t splits = attn_sm_count() / (ctas > 0 ? ctas : 1);
+  const int tiles = tiles_for(max_q, max_kv, window, tpc);
+  int64_t splits = (int64_t)sm_count() * pl.minb / (ctas > 0 ? ctas : 1);
   if (splits > tiles / 4) splits = tiles / 4;                    // a part keeps at least four key tiles
   return (int)(splits < 1 ? 1 : (splits > 32 ? 32 : splits));
 }
@@ -581,7 +611,7 @@ extern "C" int b200f_latent_attn(const void* q_lat, const void* cache, const int
   AttnParams p{page_table, table_pitch, kv_lens, seq_start, sink, tokens, heads, kv_rank, rot_dim, lat_pitch, out_pitch, window,
                scale * kLog2e, key_splits, ws, 1, heads, 1};
   const AttnPlan pl = (dtype == B200F_BF16 && !simple && lat_pitch % 8 == 0 && out_pitch % 2 == 0 && aligned16(q_lat) && aligned16(cache))
-                          ? plan_attn(max_q, heads, kv_rank, rot_dim) : AttnPlan{0, 0, 0};
+                          ? plan_attn(max_q, heads, kv_rank, rot_dim) : AttnPlan{0, 0, 0, 0, 0, 0};
   if (pl.mt == 0) {
     const size_t smem = (size_t)(2 * kv_rank + rot_dim + 128 + 8) * sizeof(float);
     B200_REQUIRE(smem <= 227 * 1024, B200_E_UNSUPPORTED, "latent_attn: kv_rank %d is too large", kv_rank);
@@ -607,22 +637,22 @@ extern "C" int b200f_latent_attn(const void* q_lat, const void* cache, const int
   const bf16 *q = (const bf16*)q_lat, *kc = (const bf16*)cache;
   bf16* o = (bf16*)out;
   int rc = B200_E_UNSUPPORTED;
-#define B200_ATTN_CASE(MT_, NK_, NC_) \
-  if (pl.mt == MT_ && pl.nk == NK_ && pl.nc16 == NC_) rc = launch_mma<MT_, NK_, NC_>(p, q, kc, o, grid, d16, st);
-  B200_ATTN_CASE(1, 64, 4)
-  B200_ATTN_CASE(1, 64, 8)
-  B200_ATTN_CASE(2, 64, 4)
-  B200_ATTN_CASE(2, 64, 8)
-  B200_ATTN_CASE(2, 32, 4)
-  B200_ATTN_CASE(2, 32, 8)
-  B200_ATTN_CASE(4, 64, 4)
-  B200_ATTN_CASE(4, 64, 8)
-  B200_ATTN_CASE(4, 64, 16)
-  B200_ATTN_CASE(4, 32, 4)
-  B200_ATTN_CASE(4, 32, 8)
-  B200_ATTN_CASE(4, 32, 16)
+#define B200_ATTN_CASE(MT_, W_, ST_, KS_, NC_, MB_) \
+  if (pl.mt == MT_ && pl.ks == KS_ && pl.nc == NC_) rc = launch_mma<MT_, W_, ST_, KS_, NC_, MB_>(p, q, kc, o, grid, d16, st);
+  B200_ATTN_VARIANTS(B200_ATTN_CASE)
 #undef B200_ATTN_CASE
   if (rc != B200_OK || key_splits == 1) return rc;
   launch_pdl(latent_merge_kernel, dim3((unsigned)(tokens * heads)), dim3(128), 0, st, p, o);
   return check_launch("latent_attn (merge)");
+}
+
+extern "C" int b200f_latent_attn_status(int* out_host, int reset) {
+  B200_REQUIRE(out_host, B200_E_NULL, "latent_attn_status: null pointer");
+  cudaError_t e = cudaMemcpyFromSymbol(out_host, g_gemm_status, sizeof(int));
+  if (e == cudaSuccess && reset) {
+    const int zero = 0;
+    e = cudaMemcpyToSymbol(g_gemm_status, &zero, sizeof(int));
+  }
+  B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "latent_attn_status: %s", cudaGetErrorString(e));
+  return B200_OK;
 }

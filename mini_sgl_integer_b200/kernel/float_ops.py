@@ -100,12 +100,14 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def check_status() -> None:
-    """Raises if a bounded wait inside a linear has expired since the last check.  Synchronises with the device."""
-    st = ctypes.c_int(0)
-    call("b200f_gemm_status", ctypes.byref(st), 1)
-    if st.value:
-        raise RuntimeError(f"a wait inside a bf16 linear expired (code {st.value}: 1 loader, 2 MMA issuer, 3 epilogue, "
-                           "4 accumulator hand-back); the step's results are not valid")
+    """Raises if a bounded wait inside a linear or the attention kernel has expired since the last check.  Synchronises
+    with the device."""
+    for name, what in (("b200f_gemm_status", "a bf16 linear"), ("b200f_latent_attn_status", "the latent attention kernel")):
+        st = ctypes.c_int(0)
+        call(name, ctypes.byref(st), 1)
+        if st.value:
+            raise RuntimeError(f"a wait inside {what} expired (code {st.value}: 1 loader, 2 MMA issuer, 3 epilogue, 4 accumulator "
+                               "hand-back, 5 copying warp, 6 consumer); the step's results are not valid")
 
 
 # ----------------------------------------------------------------------------- ends of a model
