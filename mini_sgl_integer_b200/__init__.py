@@ -8,6 +8,9 @@ sm_100a CUDA in ``libb200int.so``:
   layers               <- minisgl.layers.{norm_integer, activation_integer, rotary_integer,
                           quantization.w8a8_int8}
   attention            <- minisgl.attention (backend plug-in) and minisgl.kvcache (KV pool)
+
+A small engine, scheduler and command line (``engine``, ``__main__``) serve the integer model and Sefevik, a floating-point
+design of recurrent and latent-attention layers whose kernels are in ``libb200float.so``.
 """
 from . import _lib  # noqa: F401
 

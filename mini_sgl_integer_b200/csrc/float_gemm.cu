@@ -525,7 +525,7 @@ extern "C" int b200f_gemm_splits(int64_t m, int64_t n, int64_t k, int64_t batch,
   if (dtype != B200F_BF16 || !is_decode_size(m) || m <= 0 || n <= 0 || k <= 0 || batch <= 0) return 1;
   const int64_t blocks = batch * ((n + kFBM - 1) / kFBM), num_kb = (k + kFBK - 1) / kFBK;
   int splits = (int)(blocks < sm_count() ? sm_count() / blocks : 1);
-  splits = splits < 1 ? 1 : (splits > 8 ? 8 : splits);
+  splits = splits < 1 ? 1 : (splits > 6 ? 6 : splits);      // beyond six the consumer's reading of the parts costs more
   while (splits > 1 && num_kb / splits < 4) --splits;
   while (splits > 1 && (splits - 1) * ((num_kb + splits - 1) / splits) >= num_kb) --splits;   // no empty part
   return splits;

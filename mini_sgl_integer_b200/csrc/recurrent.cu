@@ -1,4 +1,4 @@
-// Gated linear recurrence (minGRU) over fp32 state: S_t = (1 - z_t) S_(t-1) + z_t cand_t, gates from the current token only.
+// Gated linear recurrence (minGRU) over fp32 state: S_t = (1 - z_t) S_(t-1) + z_t cand_t, the gates independent of the state.
 //
 // Prompts: one CTA per (sequence, 32 channels).  A lane owns a channel, a warp owns kSeg consecutive tokens of the current
 // stretch of kWarps * kSeg tokens.  Every warp composes its tokens' affine maps (A, B): S -> A S + B, the warps exchange the

@@ -100,10 +100,10 @@ class Engine:
         self.manager.sync()
         decode = all(len(t) == 1 for t in tokens)
         batch = Batch(reqs=list(reqs), phase="decode" if decode else "prefill")
-        flat = [(k, r.table_idx) for r in reqs for k in range(r.cached_len, r.device_len)]
-        pos = torch.tensor([k for k, _ in flat], dtype=torch.int64)
-        rows = torch.tensor([s for _, s in flat], dtype=torch.int64)
-        loc = self.manager._host[rows, pos // PAGE_SIZE] * PAGE_SIZE + pos % PAGE_SIZE
+        counts = torch.tensor([len(t) for t in tokens])
+        first = torch.tensor([r.cached_len for r in reqs]) - counts.cumsum(0) + counts
+        pos = torch.arange(int(counts.sum())) + torch.repeat_interleave(first, counts)
+        loc = self.manager.locations(torch.repeat_interleave(torch.tensor([r.table_idx for r in reqs]), counts), pos)
         host = torch.stack([torch.tensor([x for t in tokens for x in t], dtype=torch.int64), pos, loc]).to(torch.int32)
         picks, base = [], 0
         for t, w in zip(tokens, want):
@@ -112,7 +112,8 @@ class Engine:
         set_global_ctx(self.ctx, replace=True)
         if decode and self._graphs is not None:
             logits = self._graphs.run(batch, host)
-            logits = logits if picks == list(range(base)) else (logits[torch.tensor(picks, device=self.device)] if picks else None)
+            if picks != list(range(base)):
+                logits = logits[torch.tensor(picks, device=self.device)] if picks else None
         else:
             dev = host.pin_memory().to(self.device, non_blocking=True)
             batch.input_ids, batch.positions, batch.out_loc = dev[0], dev[1], dev[2]

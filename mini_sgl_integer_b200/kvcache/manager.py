@@ -27,6 +27,7 @@ class CacheManager:
         self._free_pages: List[int] = list(range(num_pages - 1, -1, -1))
         self._free_slots: List[int] = list(range(num_slots - 1, -1, -1))
         self._pages: Dict[int, Dict[int, int]] = {}              # slot -> page index in the sequence -> page id
+        self._first: Dict[int, int] = {}                         # slot -> first page index not yet given back
         pitch = max(1, -(-max_len // PAGE_SIZE))
         self._host = torch.zeros((num_slots + 1, pitch), dtype=torch.int32)
         if spare_page is not None:
@@ -54,6 +55,7 @@ class CacheManager:
             raise OutOfPages("no free request slot")
         slot = self._free_slots.pop()
         self._pages[slot] = {}
+        self._first[slot] = 0
         return slot
 
     def extend(self, slot: int, start: int, end: int) -> None:
@@ -78,13 +80,19 @@ class CacheManager:
             return
         first = max(0, length - self.window + 1) // PAGE_SIZE if self.window else length // PAGE_SIZE
         have = self._pages[slot]
-        for i in [i for i in have if i < first]:
-            self._free_pages.append(have.pop(i))
+        for i in range(self._first[slot], first):
+            if i in have:
+                self._free_pages.append(have.pop(i))
+        self._first[slot] = max(first, self._first[slot])
 
     def free(self, slot: int) -> None:
         self._free_pages.extend(self._pages.pop(slot).values())
         self._free_slots.append(slot)
         self._dirty.discard(slot)
+
+    def locations(self, slots: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+        """Cache rows (page * 16 + offset) of positions (host tensors)."""
+        return self._host[slots, positions // PAGE_SIZE] * PAGE_SIZE + positions % PAGE_SIZE
 
     def sync(self) -> None:
         """Brings the device's page table up to date (one small copy)."""

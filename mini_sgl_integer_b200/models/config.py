@@ -71,7 +71,7 @@ class LatentAttentionConfig:
     vdim: int
     kv_rank: int
     scale: float
-    window: Optional[int] = None      # a token sees itself and the window - 1 before it; None: everything before it
+    window: Optional[int] = None      # width of the causal window in keys; None: unbounded
     rot: Optional[RotarySpec] = None
     kv_from: Optional[int] = None     # layer whose latent cache is used instead of an own one
 

@@ -22,4 +22,7 @@ step, the restatement is the definition):
   linear.int32_accumulate                      exact by arithmetic
   linear.requant_q15 / absmax_to_mul_shift     parity unpinned (the reference's
                                                epilogue is a float library call)
+
+  sefevik.*                                    the floating-point design, in float64; the
+                                               restatement is the definition
 """

@@ -126,7 +126,7 @@ def latent_keys(h, mix, w, pre, eps):
 
 
 def window_mask(n, size):
-    """visible[i, j]: j is i itself or one of the size - 1 tokens before it (all tokens before it without a size)."""
+    """Causal band matrix: row i holds the last `size` keys up to i (every key up to i when size is None)."""
     i, j = np.arange(n)[:, None], np.arange(n)[None, :]
     ok = j <= i
     return ok if size is None else ok & (i - j < size)
