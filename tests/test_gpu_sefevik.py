@@ -89,6 +89,20 @@ def test_decoding_from_the_first_token(name, dtype):
     check(feed(e, r, ids, list(range(1, 90))), want, limits(name, ids, want, dtype))
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["mixed", "wide heads"])
+def test_long_prompt(name, dtype):
+    """Enough tokens per forward for the large linears, and for many stretches of the scan and key tiles."""
+    ids = np.random.default_rng(13).integers(0, CONFIGS[name]["vocab"], 640)
+    want = oracle(name, ids)
+    limit = limits(name, ids, want, dtype)
+    e = engine(name, dtype)
+    for c in ([], [300, 302, 639], [129, 257, 513]):
+        r = e.open()
+        check(feed(e, r, ids, c), want, limit)
+        e.close(r)
+
+
 @pytest.mark.parametrize("graphs", [True, False])
 def test_long_decoding_holds_no_more_pages_than_the_window(graphs):
     name, ids = "mixed", np.random.default_rng(6).integers(0, 131, 420)
