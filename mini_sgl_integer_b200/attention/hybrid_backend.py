@@ -1,4 +1,4 @@
-"""Backend of hybrid models (latent attention + recurrent state): the metadata of a batch and its CUDA-graph buffers,
+"""Backend of hybrid models (paged attention + recurrent state): the metadata of a batch and its CUDA-graph buffers,
 behind the interface of ``BaseAttnBackend``.  The mixers launch their own kernels with this metadata, so there is no
 per-layer ``forward`` on separate q, k and v."""
 from __future__ import annotations
@@ -47,7 +47,7 @@ class B200HybridBackend(BaseAttnBackend):
         return get_global_ctx().page_table
 
     def forward(self, q, k, v, layer_id, batch):
-        raise NotImplementedError("latent attention runs inside its layer (layers/latent_attention.py)")
+        raise NotImplementedError("the mixers of hybrid models run their attention inside their layers")
 
     def prepare_metadata(self, batch) -> None:
         """From ``batch.padded_reqs`` (table_idx, cached_len, device_len), ``batch.positions`` and ``batch.out_loc``."""

@@ -19,7 +19,8 @@ INCLUDE = os.path.join(os.path.dirname(PKG_DIR), "include")
 LIBRARIES = {
     "int": ("libb200int.so", ["runtime.cu", "api.cu", "batch_ops.cu", "rowops.cu", "attn.cu", "attn_split.cu", "attn_prefill.cu",
                               "gemm.cu", "model_ops.cu", "tp.cu"]),
-    "float": ("libb200float.so", ["runtime.cu", "batch_ops.cu", "float_gemm.cu", "float_rows.cu", "recurrent.cu", "latent_attn.cu"]),
+    "float": ("libb200float.so", ["runtime.cu", "batch_ops.cu", "float_gemm.cu", "float_rows.cu", "recurrent.cu", "latent_attn.cu", "matrix_memory.cu",
+                                  "grouped_attn.cu"]),
 }
 LIB_PATH = os.path.join(PKG_DIR, LIBRARIES["int"][0])
 NVCC_FLAGS = [

@@ -70,6 +70,38 @@ __device__ __forceinline__ void f_store_chunk(int* stage, int lane, int (&v)[32]
 #pragma unroll
     for (int j = 0; j < 32; ++j) v[j] = __float_as_int(xielu_f32(__int_as_float(v[j]), p.act_a, p.act_b));
   }
+  if (p.act == B200F_ACT_GATED_SILU) {       // the chunk's first 16 columns are gates, the others what they gate
+    bf16* out = reinterpret_cast<bf16*>(p.out) + boff;
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < 8; j += 4) {
+      unsigned w[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = 2 * (j + i);
+        w[i] = f32_to_bf16x2(silu_f32(__int_as_float(v[c])) * __int_as_float(v[16 + c]), silu_f32(__int_as_float(v[c + 1])) * __int_as_float(v[17 + c]));
+      }
+      *reinterpret_cast<uint4*>(stage + lane * kFStagePitch + j) = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+    __syncwarp();
+#pragma unroll
+    for (int it = 0; it < 2; ++it) {
+      const int r = it * 16 + (lane >> 1), row = r_base + r, col = (col0 >> 1) + 8 * (lane & 1), n = p.N >> 1;
+      if (row < p.M && col < n) {
+        const uint4 o = *reinterpret_cast<const uint4*>(stage + r * kFStagePitch + 4 * (lane & 1));
+        bf16* dst = out + (int64_t)row * p.out_pitch + col;
+        if (p.vec && col + 7 < n) {
+          *reinterpret_cast<uint4*>(dst) = o;
+        } else {
+          const unsigned w[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (col + i < n) reinterpret_cast<unsigned short*>(dst)[i] = (unsigned short)(w[i >> 1] >> (16 * (i & 1)));
+        }
+      }
+    }
+    return;
+  }
   const int rr = lane >> 2, cc = (lane & 3) * 4;
   if (p.out_f32) {
     float* out = reinterpret_cast<float*>(p.out) + boff;
@@ -260,7 +292,15 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           if (c0 >= p.M) break;
           int v[32];
           tmem_ld_32x32(tmem_base + ((unsigned)(q * 32) << 16) + slot * BN + (unsigned)c0, v);
-          if (ok && ch < p.N) {
+          if (p.act == B200F_ACT_GATED_SILU) {                   // weight rows alternate: 16 gates, 16 gated
+            bf16* out = reinterpret_cast<bf16*>(p.out) + (int64_t)t.b * p.out_bstride + ((ch >> 5) * 16 + (ch & 15));
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              const float up = __int_as_float(__shfl_down_sync(FULL_MASK, v[j], 16));
+              if (ok && lane < 16 && ch < p.N && c0 + j < p.M)
+                out[(int64_t)(c0 + j) * p.out_pitch] = __float2bfloat16_rn(silu_f32(__int_as_float(v[j])) * up);
+            }
+          } else if (ok && ch < p.N) {
             if (p.act == B200F_ACT_XIELU) {
 #pragma unroll
               for (int j = 0; j < 32; ++j) v[j] = __float_as_int(xielu_f32(__int_as_float(v[j]), p.act_a, p.act_b));
@@ -539,8 +579,9 @@ extern "C" int b200f_gemm(const void* x, const void* w, void* out, int dtype, in
   B200_REQUIRE(x && w && out, B200_E_NULL, "gemm: null pointer");
   B200_REQUIRE(m >= 0 && n > 0 && k > 0 && batch > 0 && m < (1ll << 31) && n < (1ll << 31) && k < (1ll << 31) && batch < (1 << 16),
                B200_E_SHAPE, "gemm: m=%lld n=%lld k=%lld batch=%lld", (long long)m, (long long)n, (long long)k, (long long)batch);
-  B200_REQUIRE(x_pitch >= k && w_pitch >= k && out_pitch >= n, B200_E_SHAPE, "gemm: a row pitch is shorter than its row");
-  B200_REQUIRE(act == B200F_ACT_NONE || act == B200F_ACT_XIELU, B200_E_UNSUPPORTED, "gemm: activation %d", act);
+  B200_REQUIRE(x_pitch >= k && w_pitch >= k && out_pitch >= (act == B200F_ACT_GATED_SILU ? n / 2 : n), B200_E_SHAPE, "gemm: a row pitch is shorter than its row");
+  B200_REQUIRE(act == B200F_ACT_NONE || act == B200F_ACT_XIELU || (act == B200F_ACT_GATED_SILU && dtype == B200F_BF16 && !out_f32 && n % 32 == 0),
+               B200_E_UNSUPPORTED, "gemm: activation %d", act);
   B200_REQUIRE(splits >= 1 && (splits == 1 || (act == B200F_ACT_NONE && out_f32 && dtype == B200F_BF16 && is_decode_size(m))),
                B200_E_UNSUPPORTED, "gemm: splits=%d needs a 32-bit output without activation at decode sizes", splits);
   if (m == 0) return B200_OK;

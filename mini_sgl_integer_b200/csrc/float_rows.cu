@@ -1,5 +1,6 @@
-// Row kernels of the floating-point models: embedding (+ bigram row), the end of a sublayer (output norm, residual add,
-// depth average, final norm), xIELU, and the arg-max over fp32 logits.  Streams, norms and averages are fp32; the
+// Row kernels of the floating-point models: embedding (+ bigram row), the end of a sublayer (mean of two normed outputs,
+// output norm, residual add, added vector, depth average, norm in front of the next linear), xIELU, gated SiLU, and the
+// arg-max over fp32 logits.  Streams, norms and averages are fp32; the
 // T-typed copies feed the next linear.
 #include "float_common.cuh"
 
@@ -63,7 +64,12 @@ struct SublayerEnd {
   const float* y;
   int splits;
   int64_t split_stride;
-  const float *x_in, *norm_w;
+  const float* y2;                   // nullable: the output is the mean of y normed with gain w1 and y2 normed with gain w2
+  int splits2;
+  int64_t split_stride2;
+  const float *w1, *w2;
+  const float *x_in, *norm_w;        // x_in nullable: zero
+  const float* add;                  // nullable: a vector for every row
   float* x_out;
   const float* hist;
   int planes;
@@ -115,26 +121,51 @@ __global__ void sublayer_end_kernel(const SublayerEnd p, T* __restrict__ x_out_t
   int col[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) col[i] = (i * blockDim.x + threadIdx.x) * VEC;
-  if (p.y) {
+  // the sum of a stack of parts and its sum of squares
+  auto take = [&](const float* y, int splits, int64_t stride, Pack<VEC> (&a)[NV]) {
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       if (col[i] >= p.width) continue;
-      r[i] = load_pack<VEC>(p.y + base + col[i]);
-      for (int s = 1; s < p.splits; ++s) {
-        const Pack<VEC> o = load_pack<VEC>(p.y + (int64_t)s * p.split_stride + base + col[i]);
+      a[i] = load_pack<VEC>(y + base + col[i]);
+      for (int s = 1; s < splits; ++s) {
+        const Pack<VEC> o = load_pack<VEC>(y + (int64_t)s * stride + base + col[i]);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) r[i].v[k] += o.v[k];
+        for (int k = 0; k < VEC; ++k) a[i].v[k] += o.v[k];
       }
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) ss = fmaf(r[i].v[k], r[i].v[k], ss);
+      for (int k = 0; k < VEC; ++k) ss = fmaf(a[i].v[k], a[i].v[k], ss);
+    }
+    return ss;
+  };
+  if (p.y) {
+    float ss = take(p.y, p.splits, p.split_stride, r);
+    if (p.y2) {
+      Pack<VEC> r2[NV];
+      const float ss2 = block_sum(take(p.y2, p.splits2, p.split_stride2, r2), scratch);
+      const float i1 = 0.5f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps), i2 = 0.5f / sqrtf(ss2 / (float)p.width + p.eps);
+      ss = 0.0f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        if (col[i] >= p.width) continue;
+        const Pack<VEC> a = load_pack<VEC>(p.w1 + col[i]), b = load_pack<VEC>(p.w2 + col[i]);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+          r[i].v[k] = fmaf(r[i].v[k] * i1, a.v[k], r2[i].v[k] * i2 * b.v[k]);
+          ss = fmaf(r[i].v[k], r[i].v[k], ss);
+        }
+      }
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       if (col[i] >= p.width) continue;
-      const Pack<VEC> x = load_pack<VEC>(p.x_in + base + col[i]), w = load_pack<VEC>(p.norm_w + col[i]);
+      Pack<VEC> x;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) x.v[k] = 0.0f;
+      if (p.x_in) x = load_pack<VEC>(p.x_in + base + col[i]);
+      const Pack<VEC> w = load_pack<VEC>(p.norm_w + col[i]);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) r[i].v[k] = fmaf(r[i].v[k] * inv, w.v[k], x.v[k]);
     }
@@ -142,6 +173,15 @@ __global__ void sublayer_end_kernel(const SublayerEnd p, T* __restrict__ x_out_t
 #pragma unroll
     for (int i = 0; i < NV; ++i)
       if (col[i] < p.width) r[i] = load_pack<VEC>(p.x_in + base + col[i]);
+  }
+  if (p.add) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      if (col[i] >= p.width) continue;
+      const Pack<VEC> a = load_pack<VEC>(p.add + col[i]);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[i].v[k] += a.v[k];
+    }
   }
   if (p.coef) {
     const float c_new = p.coef[p.planes];
@@ -228,6 +268,27 @@ xielu_kernel(const float* __restrict__ y, int splits, int64_t split_stride, T* _
   }
 }
 
+// silu(gate) * up over a stack of partial sums [rows, 2 * padded] whose columns alternate: 16 of gate, 16 of up.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_silu_kernel(const float* __restrict__ y, int splits, int64_t split_stride, int64_t y_pitch, T* __restrict__ out, int n,
+                  int64_t out_pitch, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t row = blockIdx.y;
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= n) return;
+  const float* src = y + row * y_pitch + (c >> 4) * 32 + (c & 15);
+  T* dst = out + row * out_pitch + c;
+  if (vec) {
+    const float4 g = part_sum4(src, splits, split_stride), u = part_sum4(src + 16, splits, split_stride);
+    store4(dst, make_float4(silu_f32(g.x) * u.x, silu_f32(g.y) * u.y, silu_f32(g.z) * u.z, silu_f32(g.w) * u.w));
+  } else {
+    for (int k = 0; k < 4 && c + k < n; ++k)
+      dst[k] = from_f32<T>(silu_f32(part_sum(src + k, splits, split_stride)) * part_sum(src + 16 + k, splits, split_stride));
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------
 // Arg-max of fp32 rows; the bits of a float are mapped to an unsigned that orders alike, then (value, index) is
 // packed as in the int32 arg-max.  A NaN never wins.
@@ -285,7 +346,8 @@ template <typename T>
 static int sublayer_end_typed(const SublayerEnd& p, void* x_out_t, int64_t rows, cudaStream_t st) {
   const bool vec = p.width % 4 == 0 && p.split_stride % 4 == 0 && p.plane_stride % 4 == 0 && p.t_pitch % 4 == 0 &&
                    aligned16(p.y) && aligned16(p.x_in) && aligned16(p.norm_w) && aligned16(p.x_out) && aligned16(p.hist) &&
-                   aligned16(p.hist_out) && aligned16(p.final_w) && aligned16(x_out_t);
+                   aligned16(p.hist_out) && aligned16(p.final_w) && aligned16(x_out_t) && p.split_stride2 % 4 == 0 && aligned16(p.y2) &&
+                   aligned16(p.w1) && aligned16(p.w2) && aligned16(p.add);
   return vec ? launch_sublayer_end<T, 4>(p, (T*)x_out_t, rows, st) : launch_sublayer_end<T, 1>(p, (T*)x_out_t, rows, st);
 }
 
@@ -312,18 +374,40 @@ extern "C" int b200f_embed_bigram(const void* table, const void* bigram, const i
   return check_launch("embed_bigram");
 }
 
-extern "C" int b200f_sublayer_end(const float* y, int splits, int64_t split_stride, const float* x_in, const float* norm_w,
-                                  float* x_out, void* x_out_t, const float* hist, int planes, int64_t plane_stride,
-                                  const float* coef, float* hist_out, const float* final_w, int dtype, int64_t rows,
-                                  int width, int64_t t_pitch, float eps, b200_stream_t s) {
+extern "C" int b200f_sublayer_end(const float* y, int splits, int64_t split_stride, const float* y2, int splits2,
+                                  int64_t split_stride2, const float* w1, const float* w2, const float* x_in,
+                                  const float* norm_w, const float* add, float* x_out, void* x_out_t, const float* hist,
+                                  int planes, int64_t plane_stride, const float* coef, float* hist_out, const float* final_w,
+                                  int dtype, int64_t rows, int width, int64_t t_pitch, float eps, b200_stream_t s) {
   B200_REQUIRE(valid_dtype(dtype), B200_E_UNSUPPORTED, "sublayer_end: dtype %d", dtype);
-  B200_REQUIRE(rows >= 0 && rows < (1ll << 31) && width > 0 && splits >= 1 && planes >= 0 && (!x_out_t || t_pitch >= width), B200_E_SHAPE,
+  B200_REQUIRE(rows >= 0 && rows < (1ll << 31) && width > 0 && splits >= 1 && splits2 >= 1 && planes >= 0 && (!x_out_t || t_pitch >= width), B200_E_SHAPE,
                "sublayer_end: rows=%lld width=%d splits=%d planes=%d", (long long)rows, width, splits, planes);
   if (rows == 0) return B200_OK;
-  B200_REQUIRE(x_in && (!y || norm_w) && (x_out || x_out_t) && (!coef || planes == 0 || hist), B200_E_NULL, "sublayer_end: null pointer");
-  SublayerEnd p{y, splits, split_stride, x_in, norm_w, x_out, hist, planes, plane_stride, coef, hist_out, final_w, width, t_pitch, eps};
+  B200_REQUIRE((x_in || y) && (!y || norm_w) && (!y2 || (y && w1 && w2)) && (x_out || x_out_t) && (!coef || planes == 0 || hist), B200_E_NULL,
+               "sublayer_end: null pointer");
+  SublayerEnd p{y, splits, split_stride, y2, splits2, split_stride2, w1, w2, x_in, norm_w, add, x_out, hist, planes, plane_stride, coef, hist_out,
+                final_w, width, t_pitch, eps};
   return dtype == B200F_BF16 ? sublayer_end_typed<bf16>(p, x_out_t, rows, (cudaStream_t)s)
                              : sublayer_end_typed<float>(p, x_out_t, rows, (cudaStream_t)s);
+}
+
+extern "C" int b200f_gated_silu(const float* y, int splits, int64_t split_stride, int64_t y_pitch, void* out, int dtype,
+                                int64_t rows, int n, int64_t out_pitch, b200_stream_t s) {
+  B200_REQUIRE(valid_dtype(dtype), B200_E_UNSUPPORTED, "gated_silu: dtype %d", dtype);
+  B200_REQUIRE(rows >= 0 && n > 0 && splits >= 1 && out_pitch >= n && y_pitch >= (int64_t)((n + 15) / 16) * 32, B200_E_SHAPE,
+               "gated_silu: rows=%lld n=%d splits=%d", (long long)rows, n, splits);
+  if (rows == 0) return B200_OK;
+  B200_REQUIRE(y && out, B200_E_NULL, "gated_silu: null pointer");
+  const int vec = n % 4 == 0 && split_stride % 4 == 0 && y_pitch % 4 == 0 && out_pitch % 4 == 0 && aligned16(y) && aligned16(out);
+  for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
+    const int64_t m = rows - r0 < 65535 ? rows - r0 : 65535;
+    const dim3 grid((unsigned)((n + 1023) / 1024), (unsigned)m);
+    if (dtype == B200F_BF16)
+      launch_pdl(gated_silu_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)s, y + r0 * y_pitch, splits, split_stride, y_pitch, (bf16*)out + r0 * out_pitch, n, out_pitch, vec);
+    else
+      launch_pdl(gated_silu_kernel<float>, grid, dim3(256), 0, (cudaStream_t)s, y + r0 * y_pitch, splits, split_stride, y_pitch, (float*)out + r0 * out_pitch, n, out_pitch, vec);
+  }
+  return check_launch("gated_silu");
 }
 
 extern "C" int b200f_xielu(const float* y, int splits, int64_t split_stride, void* out, int dtype, int64_t rows, int n,

@@ -29,7 +29,6 @@ __device__ __forceinline__ void mingru_gate(float zp, float up, float* a, float*
   const float cand = up >= 0.0f ? up + 0.5f : sigmoid_f32(up);
   *b = z * cand;
 }
-__device__ __forceinline__ float silu_f32(float v) { return v * sigmoid_f32(v); }
 
 template <typename T>
 __global__ void __launch_bounds__(kScanWarps * 32)

@@ -14,7 +14,9 @@ import torch
 
 from .._lib import call, ptr, query, require_cuda, stream
 
-ACT_NONE, ACT_XIELU = 0, 1
+ACT_NONE, ACT_XIELU, ACT_GATED_SILU = 0, 1, 2
+MEMORY_EXP, MEMORY_SSD, MEMORY_DELTA = 0, 1, 2
+GATE_SILU_BEFORE, GATE_SIGMOID_AFTER, GATE_SILU_AFTER = 0, 1, 2
 _CODES = {torch.float32: 0, torch.bfloat16: 1}
 
 
@@ -56,13 +58,14 @@ def _check_vec(name: str, t: torch.Tensor, n: int) -> None:
 # ----------------------------------------------------------------------------- linears
 def linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, out_f32: bool = False, act: int = ACT_NONE,
            act_a: float = 0.0, act_b: float = 0.0) -> torch.Tensor:
-    """act(x w^T) for rows x [T, k] and weight rows w [n, k]."""
+    """act(x w^T) for rows x [T, k] and weight rows w [n, k]; with ACT_GATED_SILU (bf16) the weight rows alternate, 16 gates
+    and 16 values, and the result has n / 2 columns."""
     _check_rows("x", x, x.dtype)
     _check_rows("w", w, x.dtype, x.shape[1])
     T, k = x.shape
     n = w.shape[0]
     if out is None:
-        out = rows(T, n, torch.float32 if out_f32 else x.dtype, x.device)
+        out = rows(T, n // 2 if act == ACT_GATED_SILU else n, torch.float32 if out_f32 else x.dtype, x.device)
     out_f32 = out.dtype == torch.float32
     call("b200f_gemm", ptr(x), ptr(w), ptr(out), dtype_code(x.dtype), int(out_f32), T, n, k, 1, _pitch(x), 0, _pitch(w), 0,
          _pitch(out), 0, 1, 0, act, act_a, act_b, stream())
@@ -130,15 +133,26 @@ def argmax_f32(logits: torch.Tensor) -> torch.Tensor:
 
 
 # ----------------------------------------------------------------------------- rows
-def sublayer_end(y: torch.Tensor, x_in: torch.Tensor, norm_w: torch.Tensor, eps: float, x_out: Optional[torch.Tensor],
-                 x_out_t: Optional[torch.Tensor], dtype: torch.dtype, hist: Optional[torch.Tensor] = None, planes: int = 0,
-                 coef: Optional[torch.Tensor] = None, hist_out: Optional[torch.Tensor] = None,
-                 final_w: Optional[torch.Tensor] = None) -> None:
-    """r = x_in + rmsnorm(y) * norm_w; with ``coef`` then the depth average over hist[:planes] and r (r kept in
-    ``hist_out``), with ``final_w`` then that norm on the way to ``x_out_t``.  See b200f_sublayer_end."""
-    T, width = x_in.shape
-    _check_parts("y", y, width)
-    _check_vec("norm_w", norm_w, width)
+def sublayer_end(y: Optional[torch.Tensor], x_in: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float,
+                 x_out: Optional[torch.Tensor], x_out_t: Optional[torch.Tensor], dtype: torch.dtype, hist: Optional[torch.Tensor] = None,
+                 planes: int = 0, coef: Optional[torch.Tensor] = None, hist_out: Optional[torch.Tensor] = None,
+                 final_w: Optional[torch.Tensor] = None, mean_with: Optional[tuple] = None, add: Optional[torch.Tensor] = None) -> None:
+    """r = x_in + rmsnorm(y) * norm_w (``x_in`` None: zero; ``y`` None: r = x_in), plus the vector ``add``; with ``coef``
+    then the depth average over hist[:planes] and r (r kept in ``hist_out``), with ``final_w`` then that norm on the way to
+    ``x_out_t``.  ``mean_with`` (w1, y2, w2): the mean of rmsnorm(y) * w1 and rmsnorm(y2) * w2 takes the place of y.  x_in and
+    x_out may be the same tensor.  See b200f_sublayer_end."""
+    T, width = (y.shape[1:] if x_in is None else x_in.shape)
+    if y is not None:
+        _check_parts("y", y, width)
+        _check_vec("norm_w", norm_w, width)
+    w1, y2, w2 = mean_with or (None, None, None)
+    if mean_with is not None:
+        _check_parts("y2", y2, width)
+        _check_vec("w1", w1, width)
+        _check_vec("w2", w2, width)
+    for name, t in (("add", add), ("final_w", final_w)):
+        if t is not None:
+            _check_vec(name, t, width)
     for t in (x_in, x_out, hist_out):
         if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape != (T, width)):
             raise ValueError("sublayer_end: streams must be contiguous fp32 [rows, width]")
@@ -148,8 +162,16 @@ def sublayer_end(y: torch.Tensor, x_in: torch.Tensor, norm_w: torch.Tensor, eps:
         _check_vec("coef", coef, planes + 1)
         if hist is None or hist.dtype != torch.float32 or not hist.is_contiguous() or hist.shape[0] < planes or hist.shape[1:] != (T, width):
             raise ValueError("sublayer_end: hist must be contiguous fp32 [planes, rows, width]")
-    call("b200f_sublayer_end", ptr(y), y.shape[0], T * width, ptr(x_in), ptr(norm_w), ptr(x_out), ptr(x_out_t), ptr(hist), planes, T * width,
-         ptr(coef), ptr(hist_out), ptr(final_w), dtype_code(dtype), T, width, 0 if x_out_t is None else _pitch(x_out_t), float(eps), stream())
+    call("b200f_sublayer_end", ptr(y), 1 if y is None else y.shape[0], T * width, ptr(y2), 1 if y2 is None else y2.shape[0], T * width, ptr(w1),
+         ptr(w2), ptr(x_in), ptr(norm_w), ptr(add), ptr(x_out), ptr(x_out_t), ptr(hist), planes, T * width, ptr(coef), ptr(hist_out), ptr(final_w),
+         dtype_code(dtype), T, width, 0 if x_out_t is None else _pitch(x_out_t), float(eps), stream())
+
+
+def gated_silu(y: torch.Tensor, out: torch.Tensor) -> None:
+    """silu(gate) * value over parts [parts, T, n] whose columns alternate, 16 gates and 16 values; out rows [T, <= n / 2]."""
+    _check_parts("y", y, y.shape[2])
+    call("b200f_gated_silu", ptr(y), y.shape[0], y.shape[1] * y.shape[2], y.shape[2], ptr(out), dtype_code(out.dtype), y.shape[1], out.shape[1],
+         _pitch(out), stream())
 
 
 def xielu(y: torch.Tensor, out: torch.Tensor, act_a: float, act_b: float) -> None:
@@ -207,3 +229,107 @@ def latent_attention(q_lat: torch.Tensor, cache: torch.Tensor, page_table: torch
     ws = torch.empty(floats, dtype=torch.float32, device=q_lat.device) if floats else None
     call("b200f_latent_attn", ptr(q_lat), ptr(cache), ptr(page_table), page_table.stride(0), ptr(kv_lens), ptr(seq_start), ptr(sink), ptr(out),
          code, T, batch, max_q, heads, kv_rank, rot_dim, pitch, out.shape[2], window, float(scale), key_splits, ptr(ws), int(simple), stream())
+
+
+def memory_prepare(y: torch.Tensor, col0: int, segments, conv_w: Optional[torch.Tensor], conv_b: Optional[torch.Tensor],
+                   conv_state: Optional[torch.Tensor], slots, positions, seq_start, seq_ids, out: torch.Tensor, kind: int, heads: int,
+                   gate_cols, gate_a: torch.Tensor, gate_b: torch.Tensor, gates: torch.Tensor, cap: float = 0.0,
+                   norm_state: Optional[torch.Tensor] = None) -> None:
+    """Between the projections of a matrix recurrence and its scan; see b200f_memory_prepare.  ``segments``: three pairs
+    (columns, head size); out rows of padded heads; gates fp32 [T, heads, 4]."""
+    parts, T, n = y.shape
+    _check_parts("y", y, n)
+    width, padded = sum(w for w, _ in segments), sum(w // h * pad8(h) for w, h in segments)
+    _check_rows("out", out, out.dtype, padded)
+    _check_vec("gates", gates, T * heads * 4)
+    _check_vec("gate_a", gate_a, heads)
+    _check_vec("gate_b", gate_b, heads)
+    taps = 0
+    if conv_w is not None:
+        taps = conv_w.shape[1]
+        _check_vec("conv_w", conv_w, width * taps)
+        if conv_b is not None:
+            _check_vec("conv_b", conv_b, width)
+        if taps > 1 and (conv_state.dtype != torch.float32 or conv_state.shape[1:] != (taps - 1, width) or not conv_state.is_contiguous()):
+            raise ValueError(f"conv_state must be contiguous fp32 [slots, {taps - 1}, {width}]")
+    if kind == MEMORY_EXP and (norm_state.dtype != torch.float32 or norm_state.shape[1] != heads or not norm_state.is_contiguous()):
+        raise ValueError(f"norm_state must be contiguous fp32 [slots, {heads}, dim + 1]")
+    seg = (ctypes.c_int32 * 6)(*[v for s in segments for v in s])
+    call("b200f_memory_prepare", ptr(y), parts, T * n, n, col0, ctypes.cast(seg, ctypes.c_void_p), ptr(conv_w), ptr(conv_b), taps,
+         ptr(conv_state) if taps > 1 else None, ptr(slots), ptr(positions), ptr(seq_start), ptr(seq_ids), ptr(out), _pitch(out), dtype_code(out.dtype),
+         kind, heads, gate_cols[0], gate_cols[1], ptr(gate_a), ptr(gate_b), float(cap), ptr(gates), ptr(norm_state),
+         0 if norm_state is None else norm_state.shape[2] - 1, T, slots.numel(), stream())
+
+
+def memory_scan(rows_: torch.Tensor, offsets, qk_heads: int, heads: int, dim: int, vdim: int, kind: int, gates: torch.Tensor, q_scale: float,
+                skip: Optional[torch.Tensor], state: torch.Tensor, norm_state: Optional[torch.Tensor], slots, positions, seq_start,
+                out: torch.Tensor, den: Optional[torch.Tensor]) -> None:
+    """Read-outs of a matrix recurrence; ``state`` fp32 [slots, heads, dim, round8(vdim)] is updated; see b200f_memory_scan.
+    ``offsets``: columns of the first q, k and v head; out fp32 [T, heads * vdim], den fp32 [T, heads]."""
+    T = rows_.shape[0]
+    _check_rows("rows", rows_, rows_.dtype)
+    _check_vec("gates", gates, T * heads * 4)
+    _check_vec("out", out, T * heads * vdim)
+    if state.dtype != torch.float32 or state.shape[1:] != (heads, dim, pad8(vdim)) or not state.is_contiguous():
+        raise ValueError(f"state must be contiguous fp32 [slots, {heads}, {dim}, {pad8(vdim)}]")
+    if skip is not None:
+        _check_vec("skip", skip, heads)
+    if kind == MEMORY_EXP:
+        _check_vec("den", den, T * heads)
+        if norm_state.shape[1:] != (heads, dim + 1) or not norm_state.is_contiguous():
+            raise ValueError(f"norm_state must be contiguous fp32 [slots, {heads}, {dim + 1}]")
+    call("b200f_memory_scan", ptr(rows_), dtype_code(rows_.dtype), _pitch(rows_), *offsets, qk_heads, heads, dim, vdim, kind, ptr(gates),
+         float(q_scale), ptr(skip), ptr(state), ptr(norm_state), ptr(slots), ptr(positions), ptr(seq_start), ptr(out), ptr(den), T, slots.numel(), stream())
+
+
+def memory_output(o: torch.Tensor, den: Optional[torch.Tensor], heads: int, vdim: int, group: int, y: torch.Tensor, gate_col: int, gate: int,
+                  norm_w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """Read-outs [T, heads * vdim] normed in groups, with the gate in column ``gate_col`` of y; see b200f_memory_output."""
+    T, n = out.shape
+    _check_vec("o", o, T * n)
+    _check_parts("y", y, y.shape[2])
+    _check_rows("out", out, out.dtype, heads * vdim)
+    _check_vec("norm_w", norm_w, norm_w.numel())
+    if den is not None:
+        _check_vec("den", den, T * heads)
+    call("b200f_memory_output", ptr(o), ptr(den), heads, vdim, group, ptr(y), y.shape[0], y.shape[1] * y.shape[2], y.shape[2], gate_col, gate,
+         ptr(norm_w), norm_w.numel(), float(eps), ptr(out), _pitch(out), dtype_code(out.dtype), T, stream())
+
+
+def grouped_prepare(y: torch.Tensor, cols, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float, out_loc, q: torch.Tensor,
+                    k_cache: torch.Tensor, v_cache: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    """Norms of q and k and the cache store of grouped attention; see b200f_grouped_prepare.  q [T, heads, pad8(dim)], caches
+    [pages, 16, kv_heads * pad8(size)]."""
+    parts, T, n = y.shape
+    _check_parts("y", y, n)
+    for name, w, k in (("q_norm", q_norm, heads * dim), ("k_norm", k_norm, kv_heads * dim)):
+        if w is not None:
+            _check_vec(name, w, k)
+    dp, vp = pad8(dim), pad8(vdim)
+    if q.shape != (T, heads, dp) or k_cache.shape[2] != kv_heads * dp or v_cache.shape[2] != kv_heads * vp or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
+        raise ValueError("grouped_prepare: q or the caches have other sizes or types")
+    require_cuda(q, k_cache, v_cache)
+    call("b200f_grouped_prepare", ptr(y), parts, T * n, n, cols[0], cols[1], cols[2], ptr(q_norm), ptr(k_norm), float(eps), ptr(out_loc), ptr(q),
+         ptr(k_cache), ptr(v_cache), dtype_code(q.dtype), T, heads, kv_heads, dim, vdim, dp, vp, k_cache.shape[0] * k_cache.shape[1], stream())
+
+
+def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, kv_lens, seq_start,
+                      out: torch.Tensor, kv_heads: int, dim: int, vdim: int, window: int, scale: float, max_q: int, max_kv: int,
+                      key_splits: int = 0, simple: bool = False) -> None:
+    """Attention over paged keys and values; see b200f_grouped_attn.  out rows [T, heads * vdim].  ``key_splits`` 0 lets the
+    library choose over how many CTAs a decode row's keys are spread."""
+    T, heads, dp = q.shape
+    vp = v_cache.shape[2] // kv_heads
+    if k_cache.dtype != q.dtype or v_cache.dtype != q.dtype or k_cache.shape[2] != kv_heads * dp or not (q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()):
+        raise ValueError("grouped_attention: q and the caches must be contiguous and of one dtype and pitch")
+    _check_rows("out", out, q.dtype, heads * vdim)
+    require_cuda(q, k_cache, v_cache, page_table, kv_lens)
+    code, batch = dtype_code(q.dtype), kv_lens.numel()
+    if simple:
+        key_splits = 1
+    elif key_splits <= 0:
+        key_splits = query("b200f_grouped_attn_splits", T, batch, max_q, max_kv, heads, kv_heads, dim, vdim, window, code)
+    floats = query("b200f_grouped_attn_ws_floats", T, heads, vdim, key_splits)
+    ws = torch.empty(floats, dtype=torch.float32, device=q.device) if floats else None
+    call("b200f_grouped_attn", ptr(q), ptr(k_cache), ptr(v_cache), ptr(page_table), page_table.stride(0), ptr(kv_lens), ptr(seq_start), ptr(out),
+         code, T, batch, max_q, heads, kv_heads, dim, vdim, dp, vp, _pitch(out), window, float(scale), key_splits, ptr(ws), int(simple), stream())

@@ -77,15 +77,100 @@ class LatentAttentionConfig:
 
 
 @dataclass(frozen=True)
+class MLSTMConfig:
+    """Matrix memory with exponential gates."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float                   # log gates are cap * tanh(pre / cap)
+
+
+@dataclass(frozen=True)
+class GatedDeltaConfig:
+    """Matrix memory written by the delta rule, one decay per head."""
+
+    heads: int
+    kv_heads: int                     # query / key heads
+    dim: int
+    vdim: int
+    conv: int                         # taps of the short convolutions
+
+
+@dataclass(frozen=True)
+class Mamba2Config:
+    heads: int
+    vdim: int
+    state: int
+    groups: int                       # of B and C
+    conv: int
+    norm_groups: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class GroupedAttentionConfig:
+    """Softmax attention whose query heads share key heads; q and k normed over the whole projection, no rotation."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class ParallelConfig:
+    """Two mixers that read the same input."""
+
+    left: GroupedAttentionConfig
+    right: Mamba2Config
+
+
+@dataclass(frozen=True)
 class DenseMLPConfig:
     ff: int
 
 
 @dataclass(frozen=True)
 class HybridLayerConfig:
-    type: str                         # "mingru" or "latent_attention"
+    type: str                         # "mingru", "latent_attention", "mlstm", "delta", "parallel"
     mixer: Any
     mlp: Optional[DenseMLPConfig] = None
+
+
+@dataclass(frozen=True)
+class RunMemory:
+    """What one run of a layer keeps per sequence.  ``planes``: (heads, values per head) of the rows it stores per token in
+    pages, keys first; ``value_prefix``: values are the first entries of the key row.  ``state``: name -> shape, fp32."""
+
+    planes: Tuple[Tuple[int, int], ...] = ()
+    value_prefix: Optional[int] = None
+    state: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
+
+
+def mixer_memory(m: Any) -> RunMemory:
+    pad = lambda n: (n + 7) // 8 * 8                                   # values of a head start on 16-byte boundaries
+    if isinstance(m, MinGRUConfig):
+        return RunMemory(state=(("s", (m.width,)),))
+    if isinstance(m, LatentAttentionConfig):
+        return RunMemory() if m.kv_from is not None else RunMemory(((1, m.kv_rank + m.rot_dim),), m.kv_rank)
+    if isinstance(m, GroupedAttentionConfig):
+        return RunMemory(((m.kv_heads, m.dim), (m.kv_heads, m.vdim)))
+    if isinstance(m, MLSTMConfig):
+        return RunMemory(state=(("S", (m.heads, m.dim, pad(m.vdim))), ("n", (m.heads, m.dim + 1))))
+    if isinstance(m, GatedDeltaConfig):
+        return RunMemory(state=(("S", (m.heads, m.dim, pad(m.vdim))), ("conv", (m.conv - 1, 2 * m.kv_heads * m.dim + m.heads * m.vdim))))
+    if isinstance(m, Mamba2Config):
+        return RunMemory(state=(("S", (m.heads, m.state, pad(m.vdim))), ("conv", (m.conv - 1, m.inner + 2 * m.groups * m.state))))
+    if isinstance(m, ParallelConfig):
+        a, b = mixer_memory(m.left), mixer_memory(m.right)
+        return RunMemory(a.planes + b.planes, state=a.state + b.state)
+    raise TypeError(f"no cache is known for {type(m).__name__}")
 
 
 @dataclass(frozen=True)
@@ -125,10 +210,11 @@ class SefevikConfig:
 
     @property
     def max_window(self) -> Optional[int]:
-        """Keys behind a token that some layer may still read (itself included); None when a layer has no window, 0
-        when no layer attends."""
-        windows = [self.layers[i].mixer.window for i in self.attention_layers]
-        return None if None in windows else max(windows, default=0)
+        return widest_window([self.layers[i].mixer.window for i in self.attention_layers])
+
+    @property
+    def memory(self) -> Tuple[RunMemory, ...]:
+        return tuple(mixer_memory(l.mixer) for l in self.layers)
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "SefevikConfig":
@@ -147,6 +233,81 @@ class SefevikConfig:
         big = (d.get("embedding") or {}).get("bigram")
         return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float(d["norm"]["eps"]), layers=layers,
                    bigram=BigramConfig(int(big["buckets"]), int(big["mul_prev"]), int(big["mul_cur"])) if big else None)
+
+
+def widest_window(windows) -> Optional[int]:
+    """Keys behind a token that some layer may still read (itself included); None when a layer has no window, 0 when no
+    layer attends."""
+    return None if None in windows else max(windows, default=0)
+
+
+@dataclass(frozen=True)
+class LoopConfig:
+    """Layers start .. stop - 1 run ``times`` times in a row."""
+
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    layer: int
+    begins: Optional[int] = None      # the pass of the loop that begins with this run
+
+
+@dataclass(frozen=True)
+class DerelornConfig:
+    """A stack of matrix memories and windowed attention, normed in front of and behind every sublayer; some layers may be
+    run several times."""
+
+    vocab_size: int
+    hidden_size: int
+    norm_eps: float
+    layers: Tuple[HybridLayerConfig, ...]
+    loop: Optional[LoopConfig] = None
+    architecture: str = "Derelorn"
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def runs(self) -> Tuple[LayerRun, ...]:
+        """Layers in the order of execution.  Every run has a cache and a state of its own."""
+        n, l = len(self.layers), self.loop
+        if l is None:
+            return tuple(LayerRun(i) for i in range(n))
+        passes = [LayerRun(i, t if i == l.start else None) for t in range(l.times) for i in range(l.start, l.stop)]
+        return tuple([LayerRun(i) for i in range(l.start)] + passes + [LayerRun(i) for i in range(l.stop, n)])
+
+    @property
+    def memory(self) -> Tuple[RunMemory, ...]:
+        return tuple(mixer_memory(self.layers[r.layer].mixer) for r in self.runs)
+
+    @property
+    def cache_layers(self) -> Tuple[int, ...]:
+        """Runs that own a paged cache."""
+        return tuple(i for i, m in enumerate(self.memory) if m.planes)
+
+    @property
+    def max_window(self) -> Optional[int]:
+        return widest_window([l.mixer.left.window for l in self.layers if l.type == "parallel"])
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "DerelornConfig":
+        if d.get("architecture") != "Derelorn":
+            raise ValueError(f"not a Derelorn configuration: architecture {d.get('architecture')!r}")
+        layers = tuple(_hybrid_layer(i, l) for i, l in enumerate(d["layers"]))
+        for i, l in enumerate(layers):
+            if l.type not in ("mlstm", "delta", "parallel"):
+                raise ValueError(f"layer {i}: the design has no mixer {l.type!r}")
+        loop = d.get("loop")
+        if loop:
+            loop = LoopConfig(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+            if not 0 <= loop.start < loop.stop <= len(layers) or loop.times < 1:
+                raise ValueError(f"loop over layers {loop.start} .. {loop.stop - 1}, {loop.times} times, of {len(layers)}")
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), norm_eps=float(d["norm"]["eps"]), layers=layers, loop=loop or None)
 
 
 def _rotary_spec(rot: Optional[Dict[str, Any]]) -> Optional[RotarySpec]:
@@ -171,9 +332,47 @@ def _hybrid_layer(i: int, l: Dict[str, Any]) -> HybridLayerConfig:
             raise ValueError(f"layer {i}: rotation over {mixer.rot.dims} of {mixer.rot_dim} entries")
         if mixer.window is not None and mixer.window < 1:
             raise ValueError(f"layer {i}: window {mixer.window}")
+    elif l["type"] == "mlstm":
+        mixer = MLSTMConfig(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+        if not mixer.gate_cap > 0:
+            raise ValueError(f"layer {i}: gate_cap {mixer.gate_cap}")
+    elif l["type"] == "delta":
+        mixer = GatedDeltaConfig(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
+        _check_shared(i, mixer.heads, mixer.kv_heads)
+        _check_taps(i, mixer.conv)
+    elif l["type"] == "parallel":
+        mixer = ParallelConfig(_grouped_attention(i, m["left"]), _mamba2(i, m["right"]))
     else:
         raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
     mlp = l.get("mlp")
     if mlp is not None and mlp.get("kind") != "dense":
         raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
     return HybridLayerConfig(l["type"], mixer, DenseMLPConfig(int(mlp["ff"])) if mlp is not None else None)
+
+
+def _check_shared(i: int, heads: int, shared: int) -> None:
+    if shared < 1 or heads % shared:
+        raise ValueError(f"layer {i}: {heads} heads cannot share {shared}")
+
+
+def _check_taps(i: int, taps: int) -> None:
+    if taps < 1:
+        raise ValueError(f"layer {i}: a convolution of {taps} taps")
+
+
+def _grouped_attention(i: int, m: Dict[str, Any]) -> GroupedAttentionConfig:
+    size = (m.get("mask") or {}).get("size")
+    c = GroupedAttentionConfig(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), None if size is None else int(size))
+    _check_shared(i, c.heads, c.kv_heads)
+    if c.window is not None and c.window < 1:
+        raise ValueError(f"layer {i}: window {c.window}")
+    return c
+
+
+def _mamba2(i: int, m: Dict[str, Any]) -> Mamba2Config:
+    c = Mamba2Config(int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["conv"]), int(m["norm_groups"]))
+    _check_shared(i, c.heads, c.groups)
+    _check_taps(i, c.conv)
+    if c.norm_groups < 1 or c.inner % c.norm_groups:
+        raise ValueError(f"layer {i}: {c.inner} values cannot be normed in {c.norm_groups} parts")
+    return c

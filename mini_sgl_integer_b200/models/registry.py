@@ -7,7 +7,7 @@ from typing import Any, Dict, Optional
 import torch
 
 from ..registry import Registry
-from .config import HadamardTransformConfig, ModelConfig, RotaryConfig, SefevikConfig
+from .config import DerelornConfig, HadamardTransformConfig, ModelConfig, RotaryConfig, SefevikConfig
 
 SUPPORTED_MODELS = Registry("Model architecture")
 
@@ -43,26 +43,18 @@ class ModelEntry:
         """Raises when a kernel of the last steps gave up waiting; synchronises with the device."""
 
 
-@SUPPORTED_MODELS.register("Sefevik")
-class SefevikEntry(ModelEntry):
+class HybridEntry(ModelEntry):
+    """Floating-point designs over ``HybridCache``."""
+
     dtypes = (torch.bfloat16, torch.float32)
     library = "float"
     backend = "b200_hybrid"
-
-    def parse_config(self, d):
-        return SefevikConfig.from_dict(d)
 
     def window(self, config):
         return config.max_window
 
     def needs_pages(self, config):
         return bool(config.cache_layers)
-
-    def create(self, config, weights, dtype, device, max_len):
-        from .sefevik import SefevikForCausalLM
-        model = SefevikForCausalLM(config, dtype, device, max_position=max_len)
-        model.load_state_dict(weights)
-        return model
 
     def create_cache(self, config, num_pages, num_slots, dtype, device):
         from ..kvcache.hybrid_pool import HybridCache
@@ -71,6 +63,30 @@ class SefevikEntry(ModelEntry):
     def check_status(self):
         from ..kernel.float_ops import check_status
         check_status()
+
+
+@SUPPORTED_MODELS.register("Sefevik")
+class SefevikEntry(HybridEntry):
+    def parse_config(self, d):
+        return SefevikConfig.from_dict(d)
+
+    def create(self, config, weights, dtype, device, max_len):
+        from .sefevik import SefevikForCausalLM
+        model = SefevikForCausalLM(config, dtype, device, max_position=max_len)
+        model.load_state_dict(weights)
+        return model
+
+
+@SUPPORTED_MODELS.register("Derelorn")
+class DerelornEntry(HybridEntry):
+    def parse_config(self, d):
+        return DerelornConfig.from_dict(d)
+
+    def create(self, config, weights, dtype, device, max_len):
+        from .derelorn import DerelornForCausalLM
+        model = DerelornForCausalLM(config, dtype, device)
+        model.load_state_dict(weights)
+        return model
 
 
 @SUPPORTED_MODELS.register("Qwen3ForCausalLM")

@@ -17,7 +17,6 @@ from typing import List, Optional
 
 import torch
 
-from ..core import get_global_ctx
 from ..kernel import float_ops as fo
 from ..layers.base import BaseOP, OPList, StateDict
 from ..layers.float_linear import FloatLinear, XieluMLP, padded_rows, take, take_f32
@@ -25,6 +24,7 @@ from ..layers.latent_attention import LatentAttention
 from ..layers.recurrent import MinGRU
 from ..layers.rotary_float import rotary_table
 from .config import HybridLayerConfig, SefevikConfig
+from .hybrid import HybridForCausalLM
 
 
 class SefevikLayer(BaseOP):
@@ -60,9 +60,7 @@ class SefevikLayer(BaseOP):
             fo.sublayer_end(self.mlp.forward(xt), x_mid, self.norm2, self._eps, x, xt, dtype, **end)
 
 
-class SefevikForCausalLM(BaseOP):
-    skips_empty_logits = True            # a batch whose ``logit_rows`` is empty runs without the head
-
+class SefevikForCausalLM(HybridForCausalLM):
     def __init__(self, config: SefevikConfig, dtype: torch.dtype = torch.bfloat16, device="cuda", max_position: int = 4096):
         self._config, self._dtype, self._device = config, dtype, torch.device(device)
         fo.dtype_code(dtype)
@@ -73,10 +71,6 @@ class SefevikForCausalLM(BaseOP):
                 ropes[rot] = rotary_table(rot, max_position, self._device)
         self.layers = OPList([SefevikLayer(config, l, i, ropes, dtype, self._device) for i, l in enumerate(config.layers)])
         self.head = FloatLinear(config.hidden_size, [config.vocab_size], ["head"], dtype, self._device)
-
-    @property
-    def config(self) -> SefevikConfig:
-        return self._config
 
     def load_state_dict(self, state_dict: StateDict, *, prefix: str = "", _internal: bool = False) -> None:
         c = self._config
@@ -115,17 +109,6 @@ class SefevikForCausalLM(BaseOP):
                 return None
             xt = xt_buf.index_select(0, logit_rows)[:, :c.hidden_size]
         return self.head.forward(xt, out_f32=True)
-
-    def forward(self) -> Optional[torch.Tensor]:
-        """Logits of the batch in the global context: of ``batch.logit_rows``, else of every request's last token."""
-        ctx = get_global_ctx()
-        batch = ctx.batch
-        rows = batch.logit_rows
-        if rows is None and batch.is_prefill:
-            rows = batch.attn_metadata.get_last_indices(batch.size).to(torch.int64)
-        return self.forward_tokens(batch.input_ids, batch.attn_metadata, ctx.attn_backend.kvcache, rows)
-
-    check_status = staticmethod(fo.check_status)
 
 
 def random_weights(config: SefevikConfig, seed: int, device="cpu", dtype: torch.dtype = torch.bfloat16) -> StateDict:

@@ -163,7 +163,7 @@ def test_float_entry_points_reject_bad_arguments_before_launch():
     assert code("b200f_latent_attn", one, one, one, 4, one, None, one, one, 1, 2, 2, 1, 4, 16, 8, 16, 16, 0, 1.0, 1, None, 0, None) == -2
     assert code("b200f_latent_attn", one, one, one, 4, one, None, one, one, 1, 2, 2, 1, 4, 16, 8, 24, 16, 0, 1.0, 2, None, 0, None) == -1
     assert code("b200f_latent_prepare", one, 1, 0, 64, one, one, one, 3, 9, None, 1e-5, one, one, None, 1, 2, 2, 4, 4, 8, 8, 8, 16, 0, None) == -2
-    assert code("b200f_sublayer_end", one, 0, 0, one, one, one, None, None, 0, 0, None, None, None, 1, 2, 8, 8, 1e-5, None) == -2
+    assert code("b200f_sublayer_end", one, 0, 0, None, 1, 0, None, None, one, one, None, one, None, None, 0, 0, None, None, None, 1, 2, 8, 8, 1e-5, None) == -2
     assert code("b200f_argmax", one, 2, 8, 4, one, None) == -2
 
 
