@@ -6,6 +6,7 @@ request is replayed from a CUDA graph captured per batch size (engine/graph.py:4
 """
 from __future__ import annotations
 
+import gc
 from typing import Any, Dict, List, Optional, Sequence
 
 import torch
@@ -180,8 +181,14 @@ class GraphRunner:
         torch.cuda.current_stream().wait_stream(side)
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph, pool=self.pool), e.ctx.forward_batch(batch):
-            logits = e.model.forward()
+        collects = gc.isenabled()
+        gc.disable()                                            # a graph or tensor freed by a collection would end the capture
+        try:
+            with torch.cuda.graph(graph, pool=self.pool), e.ctx.forward_batch(batch):
+                logits = e.model.forward()
+        finally:
+            if collects:
+                gc.enable()
         self.pool = self.pool or graph.pool()
         self.graphs[n] = (graph, logits)
 

@@ -57,7 +57,13 @@ CONFIGS = {
 
 
 def make_weights(cfg: dict, seed: int) -> dict:
-    return random_weights(DerelornConfig.from_dict(cfg), seed)
+    """bf16 weights; the first head of every mlstm layer writes weakly, so that its read-outs stay under the normaliser's floor
+    and are as small as the norms' eps."""
+    sd = random_weights(DerelornConfig.from_dict(cfg), seed)
+    for i, l in enumerate(cfg["layers"]):
+        if l["type"] == "mlstm":
+            sd[f"l{i}.mix.i.b"][0] -= 6.0
+    return sd
 
 
 def attention_window(cfg: dict):
