@@ -119,11 +119,13 @@ B200_API int b200f_latent_attn_status(int* out_host, int reset);   /* as b200f_g
  * Gates: columns gate_col_a / gate_col_b (+ head).  EXP: f and i, each cap * tanh((pre + bias) / cap) with biases gate_a /
  * gate_b, f then logsigmoid; norm_state fp32 [slots][heads][norm_dim + 1] holds n and, last, m, which is moved on here.
  * SSD and DELTA: dt from column a, gate_a = A_log, gate_b = dt_bias; DELTA: beta = sigmoid(column b).
- * gates fp32 [tokens][heads][4]: a, write strength, exp(-m).
+ * gates fp32 [tokens][heads][4]: log a, write strength, exp(-m).
  *
  * b200f_memory_scan: rows as written above (q_off, k_off, v_off: columns of the first heads; head h of `heads` uses q / k
  * head h / (heads / qk_heads)); q_scale multiplies q.  state fp32 [slots][heads][dim][round8(vdim)], taken as zero where the
- * first new token has position 0.  out fp32 [tokens][heads * vdim], den fp32 [tokens][heads] (EXP).  dim <= 512.
+ * first new token has position 0.  out fp32 [tokens][heads * vdim], den fp32 [tokens][heads] (EXP).  dim <= 512.  max_q: most
+ * new tokens of a sequence.  Prompts in bf16 run in chunks on the tensor cores (simple != 0: token by token); ws of
+ * b200f_memory_scan_ws_bytes bytes.  The other two entries of a token's gates may be overwritten.
  *
  * b200f_memory_output: u = o / den (den nullable); groups of `group` values of a row are divided by their root mean square
  * (eps inside) and multiplied by norm_w[column % norm_len]; the gate is the projection in column gate_col of y: silu(gate)
@@ -137,11 +139,13 @@ B200_API int b200f_memory_prepare(const float* y, int splits, int64_t split_stri
                                   int kind, int heads, int64_t gate_col_a, int64_t gate_col_b, const float* gate_a,
                                   const float* gate_b, float cap, float* gates, float* norm_state, int norm_dim,
                                   int64_t tokens, int batch, b200_stream_t s);
+B200_API size_t b200f_memory_scan_ws_bytes(int64_t tokens, int batch, int max_q, int heads, int dim, int vdim, int kind, int dtype);
 B200_API int b200f_memory_scan(const void* rows, int dtype, int64_t row_pitch, int64_t q_off, int64_t k_off, int64_t v_off,
-                               int qk_heads, int heads, int dim, int vdim, int kind, const float* gates, float q_scale,
+                               int qk_heads, int heads, int dim, int vdim, int kind, float* gates, float q_scale,
                                const float* skip, float* state, float* norm_state, const int32_t* slots,
                                const int32_t* positions, const int32_t* seq_start, float* out, float* den, int64_t tokens,
-                               int batch, b200_stream_t s);
+                               int batch, int max_q, void* ws, int simple, b200_stream_t s);
+B200_API int b200f_memory_scan_status(int* out_host, int reset);   /* as b200f_gemm_status: 7 a chunk's copies */
 B200_API int b200f_memory_output(const float* o, const float* den, int heads, int vdim, int group, const float* y, int splits,
                                  int64_t split_stride, int64_t y_pitch, int64_t gate_col, int gate, const float* norm_w,
                                  int norm_len, float eps, void* out, int64_t out_pitch, int dtype, int64_t tokens,

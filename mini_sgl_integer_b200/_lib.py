@@ -83,7 +83,9 @@ FLOAT_SIGNATURES: dict[str, list] = {
     "b200f_sublayer_end": [P, I, L, P, I, L, P, P, P, P, P, P, P, P, I, L, P, P, P, I, L, I, L, F, P],
     "b200f_gated_silu": [P, I, L, L, P, I, L, I, L, P],
     "b200f_memory_prepare": [P, I, L, L, L, P, P, P, I, P, P, P, P, P, P, L, I, I, I, L, L, P, P, F, P, P, I, L, I, P],
-    "b200f_memory_scan": [P, I, L, L, L, L, I, I, I, I, I, P, F, P, P, P, P, P, P, P, P, L, I, P],
+    "b200f_memory_scan_ws_bytes": [L, I, I, I, I, I, I, I],
+    "b200f_memory_scan": [P, I, L, L, L, L, I, I, I, I, I, P, F, P, P, P, P, P, P, P, P, L, I, I, P, I, P],
+    "b200f_memory_scan_status": [P, I],
     "b200f_memory_output": [P, P, I, I, I, P, I, L, L, L, I, P, I, F, P, L, I, L, P],
     "b200f_grouped_prepare": [P, I, L, L, L, L, L, P, P, F, P, P, P, P, I, L, I, I, I, I, I, I, L, P],
     "b200f_grouped_attn_ws_floats": [L, I, I, I],
@@ -101,7 +103,7 @@ FLOAT_SIGNATURES: dict[str, list] = {
 _SHARED = ("b200_last_error_string", "b200_decode_prepare")      # in every library
 _RESTYPES = {"b200_last_error_string": c_char_p, "b200_attn_workspace_bytes": ctypes.c_size_t,
              "b200_tp_block_bytes": ctypes.c_size_t, "b200f_latent_attn_ws_floats": ctypes.c_size_t,
-             "b200f_grouped_attn_ws_floats": ctypes.c_size_t}
+             "b200f_grouped_attn_ws_floats": ctypes.c_size_t, "b200f_memory_scan_ws_bytes": ctypes.c_size_t}
 
 _libs: dict[str, ctypes.CDLL] = {}
 

@@ -12,7 +12,8 @@
 //                         split into heads (each padded to 8 values), and the gates.  A token block per CTA, a channel (or
 //                         four) per thread with the taps in registers.  conv_state_kernel leaves the last inputs for the
 //                         sequence's next portion.
-// memory_scan_kernel      prompts: a CTA per (sequence, head, slice of columns) keeps its part of S in registers over all
+// memory_chunk_kernel     prompts in bf16, 64 tokens at a time on the tensor cores, see below.
+// memory_scan_kernel      prompts, any type and size (the 32-bit path; short portions): a CTA per (sequence, head, slice of columns) keeps its part of S in registers over all
 //                         tokens: LN lanes share a column quad, each holds R of its rows as fp32 pairs.  Tokens come
 //                         through shared memory in stages of 16.  Tokens are processed one by one in the order of the
 //                         equations, so how a prompt was cut makes no difference at all.
@@ -63,7 +64,7 @@ __device__ __forceinline__ int padded_column(const MemoryPrepare& p, int c) {
   return out;
 }
 
-// (first, second) gate of one token and head, as the scan reads them: EXP log gates (f, i), SSD (decay, dt), DELTA (decay, beta).
+// (first, second) gate of one token and head: EXP log gates (f, i), SSD (log decay, dt), DELTA (log decay, beta).
 __device__ __forceinline__ float2 memory_gates(const MemoryPrepare& p, const float* row, int h) {
   const float a = part_sum(row + p.gate_col_a + h, p.splits, p.split_stride);
   if (p.kind == B200F_MEMORY_EXP) {
@@ -72,9 +73,9 @@ __device__ __forceinline__ float2 memory_gates(const MemoryPrepare& p, const flo
     return make_float2(-softplus_f32(-f), i);
   }
   const float dt = softplus_f32(a + p.gate_b[h]);
-  const float decay = expf(-expf(p.gate_a[h]) * dt);
-  if (p.kind == B200F_MEMORY_SSD) return make_float2(decay, dt);
-  return make_float2(decay, sigmoid_f32(part_sum(row + p.gate_col_b + h, p.splits, p.split_stride)));
+  const float log_decay = -expf(p.gate_a[h]) * dt;
+  if (p.kind == B200F_MEMORY_SSD) return make_float2(log_decay, dt);
+  return make_float2(log_decay, sigmoid_f32(part_sum(row + p.gate_col_b + h, p.splits, p.split_stride)));
 }
 
 template <typename T, int VEC, int TAPS>      // TAPS 0: none, -1: any number
@@ -94,7 +95,7 @@ memory_prepare_kernel(const MemoryPrepare p, T* __restrict__ out) {
         float* ms = p.norm_state + ((int64_t)p.slots[t] * p.heads + h) * (p.norm_dim + 1) + p.norm_dim;
         const float m0 = p.positions[t] > 0 ? *ms : 0.0f, fm = g.x + m0, m = fmaxf(fm, g.y);
         *ms = m;
-        r = make_float4(expf(fm - m), expf(g.y - m), expf(-m), 0.0f);
+        r = make_float4(fm - m, expf(g.y - m), expf(-m), 0.0f);
       }
       p.gates[t * p.heads + h] = r;
     }
@@ -225,7 +226,7 @@ struct MemoryParams {
   int64_t row_pitch;
   int64_t q_off, k_off, v_off;         // columns in a row; heads are padded to 8 values
   int qk_heads, heads, dim, vdim;
-  const float4* gates;
+  float4* gates;
   float q_scale;
   const float* skip;                   // nullable, [heads]
   float* state;                        // [slots][heads][dim][pad8(vdim)]
@@ -368,9 +369,9 @@ memory_scan_kernel(const MemoryParams p, const T* __restrict__ rows) {
       if (KIND == B200F_MEMORY_DELTA) {
         sq = warp_sum(sq);
         sk = warp_sum(sk);
-        if (lane == 0) *reinterpret_cast<float4*>(sc + 4 * t) = make_float4(rg[t].x, rg[t].y, 1.0f / sqrtf(sk + kUnitEps), p.q_scale / sqrtf(sq + kUnitEps));
+        if (lane == 0) *reinterpret_cast<float4*>(sc + 4 * t) = make_float4(expf(rg[t].x), rg[t].y, 1.0f / sqrtf(sk + kUnitEps), p.q_scale / sqrtf(sq + kUnitEps));
       } else if (lane == 0) {
-        *reinterpret_cast<float4*>(sc + 4 * t) = make_float4(rg[t].x, rg[t].y, rg[t].z, p.q_scale);
+        *reinterpret_cast<float4*>(sc + 4 * t) = make_float4(expf(rg[t].x), rg[t].y, rg[t].z, p.q_scale);
       }
     }
     __syncthreads();
@@ -455,7 +456,7 @@ memory_scan_kernel(const MemoryParams p, const T* __restrict__ rows) {
   }
 }
 
-// Log gates (f, i) of a prompt batch to (exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t)); a warp per (sequence, head).
+// Log gates (f, i) of a prompt batch to (f + m_(t-1) - m_t, exp(i - m_t), exp(-m_t)); a warp per (sequence, head).
 __global__ void __launch_bounds__(32)
 running_max_kernel(const MemoryPrepare p) {
   __shared__ float2 fi[32];
@@ -481,9 +482,580 @@ running_max_kernel(const MemoryPrepare p) {
       if (t == lane) { before = m; after = nm; }
       m = nm;
     }
-    if (lane < n) p.gates[(base + lane) * p.heads + h] = make_float4(expf(g.x + before - after), expf(g.y - after), expf(-after), 0.0f);
+    if (lane < n) p.gates[(base + lane) * p.heads + h] = make_float4(g.x + before - after, expf(g.y - after), expf(-after), 0.0f);
   }
   if (lane == 0) *ms = m;
+}
+
+// ---------------------------------------------------------------------------------------------------
+// Chunks of 64 tokens.  With L_t the sum of the chunk's log decays up to token t, and S_0 the state in front of it,
+//
+//   o_t = e^(L_t) S_0^T q_t + sum_(s <= t) (q_t . k_s) e^(L_t - L_s) w_s          w_s: the written vector without the decay
+//   S   = e^(L_64) S_0 + sum_s k_s (e^(L_64 - L_s) w_s)^T
+//
+// Every exponent is <= 0.  EXP and SSD know w_s = b_s v_s.  For DELTA the written vectors U solve
+// (I + M) U = diag(beta) (V - diag(e^L) K S_0), M_ts = beta_t e^(L_t - L_s) (k_t . k_s) for s < t; delta_inverse_kernel
+// computes (I + M)^-1 for all chunks at once, so that only matrix products are left on the way from chunk to chunk.
+//
+// q, k and v are bf16.  S lives in fp32 accumulators; where S, decayed scores, U or the inverse are operands of a product,
+// they are the sum of two bf16 numbers (16 bits of fraction) and the small terms' product is left out.
+//
+// A CTA per (sequence, head, 64 columns); each of 4 warps owns 16 columns and holds S^T [16, dim] in accumulators over all
+// chunks.  With everything transposed, an accumulator tile has the layout of the left operand of the next product, so S, the
+// right-hand side and U never leave the registers; shared memory holds q, k, v, the decayed scores and the inverse, each
+// read as the right operand.  EXP: in the CTA of the first columns a fifth warp's first column is n, written by ones.
+// ---------------------------------------------------------------------------------------------------
+constexpr int kChunk = 64, kChunkWarps = 4, kChunkCols = 16 * kChunkWarps;
+constexpr int kPanel = kChunk * 128;     // bytes of 64 rows of 64 bf16 values, as TMA writes them with the 128-byte swizzle
+
+
+__device__ __forceinline__ void mm_ldsm(unsigned (&r)[4], unsigned addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mm_ldsm_t(unsigned (&r)[4], unsigned addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mm_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float exp2_fast(float v) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+// (a, b) as the sum of two pairs of bf16.
+__device__ __forceinline__ void split2(float a, float b, unsigned* hi, unsigned* lo) {
+  *hi = f32_to_bf16x2(a, b);
+  const float2 h = bf16x2_to_f32(*hi);
+  *lo = f32_to_bf16x2(a - h.x, b - h.y);
+}
+__device__ __forceinline__ void cp_async16_or_zero(unsigned dst, const void* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+
+__device__ __forceinline__ void bulk_copy(unsigned dst, const void* src, unsigned bytes, unsigned bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+
+// Orders this thread's accesses to shared memory in front of later bulk copies into it (behind a barrier).
+__device__ __forceinline__ void async_fence() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
+
+// Where a sequence's chunks lie among those of the batch.
+__device__ __forceinline__ int64_t chunk_index(int64_t first_token, int seq, int chunk) { return first_token / kChunk + seq + chunk; }
+
+__host__ __device__ constexpr int chunk_panels(int dr) { return dr <= 4 ? 1 : dr / 4; }
+__host__ __device__ constexpr size_t chunk_smem(int dr, bool delta) {
+  return (size_t)(2 * chunk_panels(dr) + (delta ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 8 + 1024;
+}
+// Byte offset of (row, col) in a panel.
+__host__ __device__ __forceinline__ int panel_at(int row, int col) { return row * 128 + ((((col >> 3) ^ row) & 7) << 4) + (col & 7) * 2; }
+
+// Inclusive sums of 64 values, two per lane (token = lane, lane + 32), by one warp.
+__device__ __forceinline__ void sum64(float& a, float& b, int lane) {
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float x = __shfl_up_sync(FULL_MASK, a, o), y = __shfl_up_sync(FULL_MASK, b, o);
+    if (lane >= o) { a += x; b += y; }
+  }
+  b += __shfl_sync(FULL_MASK, a, 31);
+}
+
+template <int KIND, int DR>
+__global__ void __launch_bounds__(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0), DR > 8 ? 1 : (DR == 8 && KIND == B200F_MEMORY_EXP ? 2 : 3))
+memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams p, const bf16* __restrict__ inverse) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  constexpr bool DELTA = KIND == B200F_MEMORY_DELTA, EXP = KIND == B200F_MEMORY_EXP;
+  constexpr int C = kChunk, NW = kChunkWarps, THREADS = NW * 32 + (EXP ? 32 : 0), DP = chunk_panels(DR);
+  // panels: q [DP], k [DP], v, then the decayed scores' low and high parts (DELTA: the high part takes the place of v, which is
+  // used up by then) and, DELTA, the inverse's high and low parts
+  const unsigned q_base = (smem_u32(smem) + 1023) & ~1023u, k_base = q_base + DP * kPanel, v_base = k_base + DP * kPanel;
+  const unsigned pl_base = v_base + kPanel, ph_base = DELTA ? v_base : pl_base + kPanel, t_base = pl_base + kPanel;
+  unsigned char* panels = smem + (q_base - smem_u32(smem));
+  float* ls = reinterpret_cast<float*>(panels + (2 * DP + (DELTA ? 4 : 3)) * kPanel);        // [C] L in units of log2
+  float *el = ls + C, *bs = el + C, *zs = bs + C, *rs = zs + C, *es = rs + C; // e^L; write strength; exp(-m) or 1 / |k|; scale of q; e^(L_64 - L) times b or 1 / |k|
+
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, col0 = slice * kChunkCols;
+  const int vp = p.vdim, k16 = p.dim >> 4, qh = h / (p.heads / p.qk_heads);
+  const unsigned bar = smem_u32(es + C);
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+  pdl_wait();
+  const int64_t t0 = p.seq_start[seq];
+  const int count = p.seq_start[seq + 1] - (int)t0;
+  if (count <= 0) return;
+  const bool has_state = p.positions[t0] > 0;
+  const bool is_n = EXP && warp == NW;                   // this warp's first column is the normaliser
+  const bool works = is_n ? slice == 0 : col0 + warp * 16 < vp;
+  const int64_t slot_head = (int64_t)p.slots[seq] * p.heads + h;
+  const int64_t q_col = p.q_off + (int64_t)qh * p.dim, k_col = p.k_off + (int64_t)qh * p.dim, v_col = p.v_off + (int64_t)h * vp + col0;
+
+  const float skip = KIND == B200F_MEMORY_SSD && p.skip ? p.skip[h] / p.q_scale : 0.0f;
+
+  // S^T: rows are columns col0 + 16 warp + g (+ 8) of S, accumulator columns its rows
+  float S[2 * DR][4];
+  const int c_lo = warp * 16 + g, c_hi = c_lo + 8;       // within the slice
+  float* st = p.state + slot_head * p.dim * vp + col0;
+  float* nst = EXP ? p.norm_state + slot_head * (p.dim + 1) : nullptr;
+#pragma unroll
+  for (int i = 0; i < 2 * DR; ++i)
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
+      float v = 0.0f;
+      if (has_state && works && d < p.dim) {
+        if (is_n) v = k < 2 && g == 0 ? nst[d] : 0.0f;
+        else if (col0 + c < vp) v = st[(int64_t)d * vp + c];
+      }
+      S[i][k] = v;
+    }
+
+  // ldmatrix addresses: rows of 128 bytes, 16-byte pieces exchanged by the row's last three bits
+  const unsigned n_row = ((lane & 7) + ((lane >> 4) << 3)) * 128, n_x = (((lane >> 3) & 1) ^ (lane & 7)) << 4;     // right operand from [n][k], left from [k][m]
+  const unsigned m_row = (lane & 15) * 128, m_x = ((lane >> 4) ^ (lane & 7)) << 4;                                 // left operand from [m][k], right from [k][n]
+  auto at_n = [&](unsigned base, int row16, int k16th) { return base + (k16th >> 2) * kPanel + row16 * 2048 + n_row + (n_x ^ ((k16th & 3) << 5)); };
+  auto at_m = [&](unsigned base, int row16, int k16th) { return base + (k16th >> 2) * kPanel + row16 * 2048 + m_row + (m_x ^ ((k16th & 3) << 5)); };
+
+  // acc [16 columns, 64 tokens] = S^T X^T for X = q or k
+  auto state_times = [&](unsigned x_base, float (&acc)[8][4]) {
+#pragma unroll
+    for (int kk = 0; kk < DR; ++kk) {
+      if (kk >= k16) break;
+      unsigned ah[4], al[4];
+      split2(S[2 * kk][0], S[2 * kk][1], &ah[0], &al[0]);
+      split2(S[2 * kk][2], S[2 * kk][3], &ah[1], &al[1]);
+      split2(S[2 * kk + 1][0], S[2 * kk + 1][1], &ah[2], &al[2]);
+      split2(S[2 * kk + 1][2], S[2 * kk + 1][3], &ah[3], &al[3]);
+      unsigned b[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) mm_ldsm(b[j], at_n(x_base, j, kk));
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mm_mma(acc[2 * j], ah, b[j][0], b[j][1]);
+        mm_mma(acc[2 * j + 1], ah, b[j][2], b[j][3]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mm_mma(acc[2 * j], al, b[j][0], b[j][1]);
+        mm_mma(acc[2 * j + 1], al, b[j][2], b[j][3]);
+      }
+    }
+  };
+  // V^T of 16 tokens as a left operand; in the accumulator layout: pairs of tokens
+  auto values = [&](int kb, unsigned (&a)[4]) {
+    if (is_n) {
+      a[0] = a[2] = g == 0 ? 0x3f803f80u : 0u;           // ones
+      a[1] = a[3] = 0u;
+    } else {
+      mm_ldsm_t(a, at_n(v_base, kb, warp));
+    }
+  };
+
+  const int chunks = (count + C - 1) / C;
+  float4 gate_a, gate_b;                                  // warp 0: the next chunk's gates
+  auto load_gates = [&](int ch) {
+    const float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const float4* src = p.gates + (t0 + (int64_t)ch * C + lane) * p.heads + h;
+    gate_a = ch * C + lane < count ? src[0] : z;
+    gate_b = ch * C + lane + 32 < count ? src[(int64_t)32 * p.heads] : z;
+  };
+  if (warp == 0) load_gates(0);
+  for (int ch = 0; ch < chunks; ++ch) {
+    const int n = min(C, count - ch * C);
+    const int64_t tok = t0 + (int64_t)ch * C;
+    if (warp == 0) {
+      if (lane == 0) {
+        mbar_expect_tx(bar, (2 * DP + 1) * kPanel + (DELTA ? 2 * kPanel : 0));
+#pragma unroll
+        for (int d = 0; d < DP; ++d) {
+          tma_load_2d(q_base + d * kPanel, &map, (int)q_col + 64 * d, (int)tok, bar);
+          tma_load_2d(k_base + d * kPanel, &map, (int)k_col + 64 * d, (int)tok, bar);
+        }
+        tma_load_2d(v_base, &map, (int)v_col, (int)tok, bar);
+        if (DELTA) bulk_copy(t_base, inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C), 2 * kPanel, bar);
+      }
+      __syncwarp();
+      const float4 ga = gate_a, gb = gate_b;
+      load_gates(ch + 1);
+      float la = ga.x * 1.4426950408889634f, lb = gb.x * 1.4426950408889634f;
+      sum64(la, lb, lane);
+      const float last = __shfl_sync(FULL_MASK, lb, 31);
+      ls[lane] = la; ls[lane + 32] = lb;
+      el[lane] = exp2_fast(la); el[lane + 32] = exp2_fast(lb);
+      bs[lane] = ga.y; bs[lane + 32] = gb.y;
+      zs[lane] = ga.z; zs[lane + 32] = gb.z;
+      rs[lane] = DELTA ? ga.w : p.q_scale; rs[lane + 32] = DELTA ? gb.w : p.q_scale;
+      es[lane] = exp2_fast(last - la) * (DELTA ? ga.z : ga.y); es[lane + 32] = exp2_fast(last - lb) * (DELTA ? gb.z : gb.y);
+    }
+    if (__syncthreads_or(!mbar_wait(bar, ch & 1, 7))) {    // expired (the status word says so): once more for the copies, and out
+      mbar_wait(bar, ch & 1, 7);
+      return;
+    }
+    if (n < C) {                                          // behind the portion: k and v of other sequences, to be zero here
+      for (int i = tid; i < (C - n) * 8 * (DP + 1); i += THREADS) {
+        const int r = n + i / (8 * (DP + 1)), c = i % (8 * (DP + 1));
+        *reinterpret_cast<uint4*>(panels + (DP + (c >> 3)) * kPanel + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+      }
+      __syncthreads();
+    }
+
+    float u[8][4];                                        // DELTA: U^T
+    if (DELTA) {
+      if (works) {
+        float r[8][4] = {};                               // right-hand side beta (v - e^L K S_0), transposed
+        state_times(k_base, r);
+#pragma unroll
+        for (int kb = 0; kb < 4; ++kb) {
+          unsigned v[4];
+          values(kb, v);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int t = kb * 16 + 8 * i + q2;
+            const float2 x = bf16x2_to_f32(v[2 * i]), y = bf16x2_to_f32(v[2 * i + 1]);
+            const float2 b = *reinterpret_cast<const float2*>(bs + t), e = *reinterpret_cast<const float2*>(el + t), z = *reinterpret_cast<const float2*>(zs + t);
+            const float b0 = b.x, b1 = b.y, f0 = e.x * z.x, f1 = e.y * z.y;
+            float* a = r[2 * kb + i];
+            a[0] = b0 * (x.x - f0 * a[0]); a[1] = b1 * (x.y - f1 * a[1]);
+            a[2] = b0 * (y.x - f0 * a[2]); a[3] = b1 * (y.y - f1 * a[3]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) u[i][k] = 0.0f;
+#pragma unroll
+        for (int kb = 0; kb < 4; ++kb) {
+          unsigned ah[4], al[4];
+          split2(r[2 * kb][0], r[2 * kb][1], &ah[0], &al[0]);
+          split2(r[2 * kb][2], r[2 * kb][3], &ah[1], &al[1]);
+          split2(r[2 * kb + 1][0], r[2 * kb + 1][1], &ah[2], &al[2]);
+          split2(r[2 * kb + 1][2], r[2 * kb + 1][3], &ah[3], &al[3]);
+          unsigned bh[4][4], bl[4][4];
+#pragma unroll
+          for (int j = kb; j < 4; ++j) {
+            mm_ldsm(bh[j], at_n(t_base, j, kb));
+            mm_ldsm(bl[j], at_n(t_base + kPanel, j, kb));
+          }
+#pragma unroll
+          for (int j = kb; j < 4; ++j) {
+            mm_mma(u[2 * j], ah, bh[j][0], bh[j][1]);
+            mm_mma(u[2 * j + 1], ah, bh[j][2], bh[j][3]);
+          }
+#pragma unroll
+          for (int j = kb; j < 4; ++j) {
+            mm_mma(u[2 * j], al, bh[j][0], bh[j][1]);
+            mm_mma(u[2 * j + 1], al, bh[j][2], bh[j][3]);
+          }
+#pragma unroll
+          for (int j = kb; j < 4; ++j) {
+            mm_mma(u[2 * j], ah, bl[j][0], bl[j][1]);
+            mm_mma(u[2 * j + 1], ah, bl[j][2], bl[j][3]);
+          }
+        }
+      }
+      __syncthreads();                                    // the values' place is taken by the scores
+    }
+
+    // decayed scores: the ten 16 x 16 blocks on and below the diagonal
+    constexpr int WARPS = THREADS / 32, MINE = (10 + WARPS - 1) / WARPS;
+    float sc[MINE][2][4];
+#pragma unroll
+    for (int m = 0; m < MINE; ++m)
+#pragma unroll
+      for (int k = 0; k < 8; ++k) sc[m][k >> 2][k & 3] = 0.0f;
+#pragma unroll
+    for (int kk = 0; kk < DR; ++kk) {
+      if (kk >= k16) break;
+      unsigned a[MINE][4], b[MINE][4];
+#pragma unroll
+      for (int m = 0; m < MINE; ++m) {
+        const int blk = min(warp + m * WARPS, 9), rb = (blk >= 1) + (blk >= 3) + (blk >= 6), kb = blk - rb * (rb + 1) / 2;
+        mm_ldsm(a[m], at_m(q_base, rb, kk));
+        mm_ldsm(b[m], at_n(k_base, kb, kk));
+      }
+#pragma unroll
+      for (int m = 0; m < MINE; ++m) {
+        mm_mma(sc[m][0], a[m], b[m][0], b[m][1]);
+        mm_mma(sc[m][1], a[m], b[m][2], b[m][3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MINE; ++m) {
+      const int blk = warp + m * WARPS;
+      if (blk >= 10) break;
+      const int rb = (blk >= 1) + (blk >= 3) + (blk >= 6), kb = blk - rb * (rb + 1) / 2;
+      float (&s)[2][4] = sc[m];
+      const int ra = rb * 16 + g;
+      const float la = ls[ra], lb = ls[ra + 8];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int c = kb * 16 + 8 * i + q2;
+        const float2 l = *reinterpret_cast<const float2*>(ls + c), w = *reinterpret_cast<const float2*>((DELTA ? zs : bs) + c);
+        const float l0 = l.x, l1 = l.y, w0 = w.x, w1 = w.y;
+        float s0 = s[i][0] * exp2_fast(la - l0) * w0, s1 = s[i][1] * exp2_fast(la - l1) * w1;
+        float s2 = s[i][2] * exp2_fast(lb - l0) * w0, s3 = s[i][3] * exp2_fast(lb - l1) * w1;
+        s0 = c <= ra ? s0 : 0.0f;
+        s1 = c < ra ? s1 : 0.0f;
+        s2 = c <= ra + 8 ? s2 : 0.0f;
+        s3 = c < ra + 8 ? s3 : 0.0f;
+        unsigned hi, lo;
+        split2(s0, s1, &hi, &lo);
+        unsigned char* at = panels + ra * 128 + (((kb * 2 + i) ^ g) << 4) + 2 * q2;     // (row ra + 8 has the same last bits)
+        *reinterpret_cast<unsigned*>(at + (ph_base - q_base)) = hi;
+        *reinterpret_cast<unsigned*>(at + (pl_base - q_base)) = lo;
+        split2(s2, s3, &hi, &lo);
+        *reinterpret_cast<unsigned*>(at + (ph_base - q_base) + 8 * 128) = hi;
+        *reinterpret_cast<unsigned*>(at + (pl_base - q_base) + 8 * 128) = lo;
+      }
+    }
+    __syncthreads();
+
+    if (works) {
+      float o[8][4] = {};
+      state_times(q_base, o);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float2 e = *reinterpret_cast<const float2*>(el + i * 8 + q2);
+        o[i][0] *= e.x; o[i][1] *= e.y; o[i][2] *= e.x; o[i][3] *= e.y;
+      }
+      const float decay = el[C - 1];
+#pragma unroll
+      for (int i = 0; i < 2 * DR; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) S[i][k] *= decay;
+#pragma unroll
+      for (int kb = 0; kb < 4; ++kb) {
+        // the written vectors of 16 tokens: bare for the read-outs of this chunk, decayed to its end for the state
+        unsigned wh[4], wl[4], dh[4], dl[4];
+        const float2 e0 = *reinterpret_cast<const float2*>(es + kb * 16 + q2), e1 = *reinterpret_cast<const float2*>(es + kb * 16 + 8 + q2);
+        if (DELTA) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float* x = &u[2 * kb + (i >> 1)][2 * (i & 1)];
+            const float2 e = i < 2 ? e0 : e1;
+            split2(x[0], x[1], &wh[i], &wl[i]);
+            split2(x[0] * e.x, x[1] * e.y, &dh[i], &dl[i]);
+          }
+        } else {
+          values(kb, wh);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float2 x = bf16x2_to_f32(wh[i]), e = i < 2 ? e0 : e1;
+            split2(x.x * e.x, x.y * e.y, &dh[i], &dl[i]);
+            if (KIND == B200F_MEMORY_SSD) {
+              float* y = &o[2 * kb + (i >> 1)][2 * (i & 1)];
+              y[0] = fmaf(skip, x.x, y[0]);
+              y[1] = fmaf(skip, x.y, y[1]);
+            }
+          }
+        }
+        unsigned bh[4][4], bl[4][4];
+#pragma unroll
+        for (int j = kb; j < 4; ++j) {
+          mm_ldsm(bh[j], at_n(ph_base, j, kb));
+          mm_ldsm(bl[j], at_n(pl_base, j, kb));
+        }
+#pragma unroll
+        for (int j = kb; j < 4; ++j) {
+          mm_mma(o[2 * j], wh, bh[j][0], bh[j][1]);
+          mm_mma(o[2 * j + 1], wh, bh[j][2], bh[j][3]);
+        }
+        if (DELTA) {
+#pragma unroll
+          for (int j = kb; j < 4; ++j) {
+            mm_mma(o[2 * j], wl, bh[j][0], bh[j][1]);
+            mm_mma(o[2 * j + 1], wl, bh[j][2], bh[j][3]);
+          }
+        }
+#pragma unroll
+        for (int j = kb; j < 4; ++j) {
+          mm_mma(o[2 * j], wh, bl[j][0], bl[j][1]);
+          mm_mma(o[2 * j + 1], wh, bl[j][2], bl[j][3]);
+        }
+        constexpr int KG = DR < 4 ? DR : 4;
+#pragma unroll
+        for (int k0 = 0; k0 < DR; k0 += KG) {
+          if (k0 >= k16) break;
+          unsigned b[KG][4];
+#pragma unroll
+          for (int i = 0; i < KG; ++i) mm_ldsm_t(b[i], at_m(k_base, kb, k0 + i));
+#pragma unroll
+          for (int i = 0; i < KG; ++i) {
+            mm_mma(S[2 * (k0 + i)], dh, b[i][0], b[i][1]);
+            mm_mma(S[2 * (k0 + i) + 1], dh, b[i][2], b[i][3]);
+          }
+#pragma unroll
+          for (int i = 0; i < KG; ++i) {
+            mm_mma(S[2 * (k0 + i)], dl, b[i][0], b[i][1]);
+            mm_mma(S[2 * (k0 + i) + 1], dl, b[i][2], b[i][3]);
+          }
+        }
+      }
+      if (is_n) {
+        if (g == 0) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+              const int t = i * 8 + q2 + k;
+              if (t < n) p.den[(tok + t) * p.heads + h] = fmaxf(fabsf(o[i][k] * rs[t]), zs[t]) + kUnitEps;
+            }
+        }
+      } else {
+        const int64_t pitch = (int64_t)p.heads * p.vdim;
+        float* out = p.out + (tok + q2) * pitch + (int64_t)h * p.vdim + col0 + c_lo;
+        const bool lo = col0 + c_lo < vp, hi = col0 + c_hi < vp;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float2 r = *reinterpret_cast<const float2*>(rs + i * 8 + q2);
+          const bool t_a = i * 8 + q2 < n, t_b = i * 8 + q2 + 1 < n;
+          if (t_a && lo) out[0] = o[i][0] * r.x;
+          if (t_b && lo) out[pitch] = o[i][1] * r.y;
+          if (t_a && hi) out[8] = o[i][2] * r.x;
+          if (t_b && hi) out[pitch + 8] = o[i][3] * r.y;
+          out += 8 * pitch;
+        }
+      }
+    }
+    async_fence();
+    __syncthreads();                                       // everything in shared memory may be replaced
+  }
+  if (!works) return;
+#pragma unroll
+  for (int i = 0; i < 2 * DR; ++i)
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
+      if (d >= p.dim) continue;
+      if (is_n) {
+        if (k < 2 && g == 0) nst[d] = S[i][k];
+      } else if (col0 + c < vp) {
+        st[(int64_t)d * vp + c] = S[i][k];
+      }
+    }
+}
+
+// (I + M)^-1 of every chunk and head, as two bf16 panels, and the unit factors of k and q into the gates.
+// A CTA of 4 warps per (chunk, q / k head): k . k on the tensor cores, then a pair of warps per head, a column per thread.
+__global__ void __launch_bounds__(128)
+delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* __restrict__ inverse) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  constexpr int C = kChunk;
+  const int lk = ((p.dim + 15) & ~15) + 8, k16 = (p.dim + 15) >> 4;
+  float* gm = reinterpret_cast<float*>(smem);            // [C][C] k_t . k_s
+  float* mm = gm + C * C;                                // [2][C][C] M of two heads
+  float* lsum = mm + 2 * C * C;                          // [2][C]
+  float* rk = lsum + 2 * C;                              // [C]
+  float* rq = rk + C;                                    // [C]
+  bf16* ks = reinterpret_cast<bf16*>(rq + C);            // [C][lk]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int ch = blockIdx.x, qh = blockIdx.y, seq = blockIdx.z;
+  const int64_t t0 = p.seq_start[seq];
+  const int count = p.seq_start[seq + 1] - (int)t0;
+  if (ch * C >= count) return;
+  const int n = min(C, count - ch * C), cq = p.dim / 8;
+  const int64_t tok = t0 + (int64_t)ch * C;
+  const bf16* q_src = rows + tok * p.row_pitch + p.q_off + (int64_t)qh * p.dim;
+  const bf16* k_src = rows + tok * p.row_pitch + p.k_off + (int64_t)qh * p.dim;
+  for (int i = tid; i < C * cq; i += 128) {
+    const int t = i / cq, c = (i - t * cq) * 8;
+    cp_async16_or_zero(smem_u32(ks + t * lk + c), k_src + (t < n ? t : 0) * p.row_pitch + c, t < n);
+  }
+  cp_async_commit();
+  for (int r = tid; r < C; r += 128)
+    for (int c = p.dim; c < lk; ++c) ks[r * lk + c] = __float2bfloat16_rn(0.0f);
+  for (int t = warp; t < C; t += 4) {
+    float ss = 0.0f;
+    if (t < n)
+      for (int c = lane * 2; c < p.dim; c += 64) {
+        const float2 x = bf16x2_to_f32(*reinterpret_cast<const unsigned*>(q_src + (int64_t)t * p.row_pitch + c));
+        ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
+      }
+    ss = warp_sum(ss);
+    if (lane == 0) rq[t] = p.q_scale / sqrtf(ss + kUnitEps);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  for (int kb = 0; kb <= warp; ++kb) {
+    float s[2][4] = {};
+    for (int kk = 0; kk < k16; ++kk) {
+      unsigned a[4], b[4];
+      mm_ldsm(a, smem_u32(ks + (warp * 16 + (lane & 15)) * lk + (lane >> 4) * 8 + kk * 16));
+      mm_ldsm(b, smem_u32(ks + (kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * lk + ((lane >> 3) & 1) * 8 + kk * 16));
+      mm_mma(s[0], a, b[0], b[1]);
+      mm_mma(s[1], a, b[2], b[3]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = kb * 16 + 8 * i + q2;
+      *reinterpret_cast<float2*>(gm + (warp * 16 + g) * C + c) = make_float2(s[i][0], s[i][1]);
+      *reinterpret_cast<float2*>(gm + (warp * 16 + g + 8) * C + c) = make_float2(s[i][2], s[i][3]);
+    }
+  }
+  __syncthreads();
+  if (tid < C) rk[tid] = 1.0f / sqrtf(gm[tid * C + tid] + kUnitEps);
+  const int per = p.heads / p.qk_heads, wp = warp >> 1, j = tid & 63;
+  float *m = mm + wp * C * C, *l = lsum + wp * C;
+  for (int e0 = 0; e0 < per; e0 += 2) {
+    const int h = qh * per + e0 + wp;
+    const bool live = e0 + wp < per;
+    __syncthreads();                                     // the factors are there; the last heads' M is no longer read
+    float beta = 0.0f;
+    if (live) {
+      const int64_t gi = (tok + (j < n ? j : 0)) * p.heads + h;
+      const float4 gate = j < n ? p.gates[gi] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      beta = gate.y;
+      if (j < n) {
+        p.gates[gi].z = rk[j];
+        p.gates[gi].w = rq[j];
+      }
+      if ((warp & 1) == 0) {
+        float a = gate.x, b = lane + 32 < n ? p.gates[(tok + lane + 32) * p.heads + h].x : 0.0f;
+        sum64(a, b, lane);
+        l[lane] = a * 1.4426950408889634f;
+        l[lane + 32] = b * 1.4426950408889634f;
+      }
+    }
+    __syncthreads();
+    if (live) {                                          // row j of M
+      const float lj = l[j], f = beta * rk[j];
+      for (int s = 0; s < C; ++s) {
+        const int c = (s + j) & 63;                      // rows start at different banks
+        m[j * C + c] = c < j ? f * rk[c] * gm[j * C + c] * exp2_fast(lj - l[c]) : 0.0f;
+      }
+    }
+    __syncthreads();
+    if (live) {                                          // column j of the inverse, row by row
+      unsigned char* dst = reinterpret_cast<unsigned char*>(inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C));
+      float x[C];
+#pragma unroll
+      for (int t = 0; t < C; ++t) {
+        float a0 = t == j ? 1.0f : 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
+#pragma unroll
+        for (int s = 0; s < t; s += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(m + t * C + s);
+          a0 = fmaf(-v.x, x[s], a0);
+          if (s + 1 < t) a1 = fmaf(-v.y, x[s + 1], a1);
+          if (s + 2 < t) a2 = fmaf(-v.z, x[s + 2], a2);
+          if (s + 3 < t) a3 = fmaf(-v.w, x[s + 3], a3);
+        }
+        x[t] = (a0 + a1) + (a2 + a3);
+        const bf16 hi = __float2bfloat16_rn(x[t]);
+        bf16* at = reinterpret_cast<bf16*>(dst + panel_at(t, j));
+        at[0] = hi;
+        at[C * C] = __float2bfloat16_rn(x[t] - __bfloat162float(hi));
+      }
+    }
+  }
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -518,6 +1090,7 @@ memory_step_kernel(const MemoryParams p, const T* __restrict__ rows, int vq) {
     sk = fmaf(k, k, sk);
   }
   float4 g = p.gates[(int64_t)seq * p.heads + h];
+  g.x = expf(g.x);
   g.w = p.q_scale;
   if (KIND == B200F_MEMORY_DELTA) {
     g.w = p.q_scale / sqrtf(block_sum(sq, scratch) + kUnitEps);
@@ -703,6 +1276,44 @@ static int launch_scan_shape(MemoryParams p, const T* rows, int batch, cudaStrea
   launch_pdl(memory_scan_kernel<T, KIND, LN, R>, grid, dim3(32 * warps + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, p, rows);
   return check_launch("memory_scan");
 }
+template <int KIND, int DR>
+static int launch_chunk_shape(const CUtensorMap& map, const MemoryParams& p, const bf16* inverse, int batch, cudaStream_t st) {
+  constexpr size_t bytes = chunk_smem(DR, KIND == B200F_MEMORY_DELTA);
+  static_assert(bytes <= 227 * 1024, "shared memory budget");
+  cudaError_t e = cudaFuncSetAttribute(memory_chunk_kernel<KIND, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+  B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
+  const dim3 grid((unsigned)((p.vdim + kChunkCols - 1) / kChunkCols), (unsigned)p.heads, (unsigned)batch);
+  launch_pdl(memory_chunk_kernel<KIND, DR>, grid, dim3(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, map, p, inverse);
+  return check_launch("memory_scan (chunks)");
+}
+template <int KIND>
+static int launch_chunks(const MemoryParams& p, const bf16* rows, bf16* inverse, int64_t tokens, int batch, int max_q, cudaStream_t st) {
+  CUtensorMap map;
+  {
+    EncodeTiledFn fn = encode_fn();
+    const cuuint64_t dims[2] = {(cuuint64_t)p.row_pitch, (cuuint64_t)tokens};
+    const cuuint64_t strides[1] = {(cuuint64_t)p.row_pitch * 2};
+    const cuuint32_t box[2] = {64, (cuuint32_t)kChunk}, estr[2] = {1, 1};
+    B200_REQUIRE(fn && fn(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(rows), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                          CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS,
+                 B200_E_CUDA, "memory_scan: cuTensorMapEncodeTiled failed");
+  }
+  if (KIND == B200F_MEMORY_DELTA) {
+    const size_t bytes = (size_t)3 * kChunk * kChunk * 4 + 4 * kChunk * 4 + (size_t)kChunk * (((p.dim + 15) & ~15) + 8) * 2;
+    cudaError_t e = cudaFuncSetAttribute(delta_inverse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
+    launch_pdl(delta_inverse_kernel, dim3((unsigned)((max_q + kChunk - 1) / kChunk), (unsigned)p.qk_heads, (unsigned)batch), dim3(128), bytes, st, p, rows, inverse);
+    const int rc = check_launch("memory_scan (inverse)");
+    if (rc != B200_OK) return rc;
+  }
+  if (p.dim <= 32) return launch_chunk_shape<KIND, 2>(map, p, inverse, batch, st);
+  if (p.dim <= 64) return launch_chunk_shape<KIND, 4>(map, p, inverse, batch, st);
+  if (p.dim <= 128) return launch_chunk_shape<KIND, 8>(map, p, inverse, batch, st);
+  return launch_chunk_shape<KIND, 16>(map, p, inverse, batch, st);
+}
+// The chunk form: bf16 heads of whole 16-value pieces (q, k) and without padding (v), and portions that fill a good part of a chunk.
+static bool chunks_fit(int dtype, int dim, int vdim, int max_q) { return dtype == B200F_BF16 && dim <= 256 && dim % 16 == 0 && vdim % 8 == 0 && max_q > 16; }
+
 template <typename T, int KIND>
 static int launch_scan(const MemoryParams& p, const T* rows, int batch, cudaStream_t st) {
   if (p.seq_start) {
@@ -773,14 +1384,19 @@ extern "C" int b200f_memory_prepare(const float* y, int splits, int64_t split_st
   return dtype == B200F_BF16 ? launch_prepare(p, (bf16*)out, batch, (cudaStream_t)s) : launch_prepare(p, (float*)out, batch, (cudaStream_t)s);
 }
 
+extern "C" size_t b200f_memory_scan_ws_bytes(int64_t tokens, int batch, int max_q, int heads, int dim, int vdim, int kind, int dtype) {
+  if (kind != B200F_MEMORY_DELTA || !chunks_fit(dtype, dim, vdim, max_q)) return 0;
+  return (size_t)(tokens / kChunk + batch + 1) * heads * 2 * kChunk * kChunk * sizeof(bf16);
+}
+
 extern "C" int b200f_memory_scan(const void* rows, int dtype, int64_t row_pitch, int64_t q_off, int64_t k_off, int64_t v_off,
-                                 int qk_heads, int heads, int dim, int vdim, int kind, const float* gates, float q_scale,
+                                 int qk_heads, int heads, int dim, int vdim, int kind, float* gates, float q_scale,
                                  const float* skip, float* state, float* norm_state, const int32_t* slots,
                                  const int32_t* positions, const int32_t* seq_start, float* out, float* den, int64_t tokens,
-                                 int batch, b200_stream_t s) {
+                                 int batch, int max_q, void* ws, int simple, b200_stream_t s) {
   B200_REQUIRE(valid_dtype(dtype) && valid_kind(kind), B200_E_UNSUPPORTED, "memory_scan: dtype %d, kind %d", dtype, kind);
   B200_REQUIRE(tokens >= 0 && tokens < (1ll << 31) && batch >= 0 && batch < 65536 && heads > 0 && heads < 65536 && qk_heads > 0 &&
-                   heads % qk_heads == 0 && dim > 0 && vdim > 0 && (seq_start || tokens == batch),
+                   heads % qk_heads == 0 && dim > 0 && vdim > 0 && max_q > 0 && (seq_start || tokens == batch),
                B200_E_SHAPE, "memory_scan: tokens=%lld batch=%d heads=%d/%d dim=%d vdim=%d", (long long)tokens, batch, heads, qk_heads, dim, vdim);
   B200_REQUIRE(dim <= 512, B200_E_UNSUPPORTED, "memory_scan: dim %d is above 512", dim);
   const int64_t hq = (dim + 7) & ~7, vp = (vdim + 7) & ~7;
@@ -790,10 +1406,30 @@ extern "C" int b200f_memory_scan(const void* rows, int dtype, int64_t row_pitch,
   B200_REQUIRE(rows && gates && state && slots && positions && out && (kind != B200F_MEMORY_EXP || (norm_state && den)), B200_E_NULL, "memory_scan: null pointer");
   B200_REQUIRE(aligned16(rows) && aligned16(gates) && aligned16(state) && row_pitch % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0,
                B200_E_ALIGN, "memory_scan: rows and heads must start on 16-byte boundaries");
-  MemoryParams p{row_pitch, q_off, k_off, v_off, qk_heads, heads, dim, vdim, reinterpret_cast<const float4*>(gates), q_scale, skip, state, norm_state,
+  MemoryParams p{row_pitch, q_off, k_off, v_off, qk_heads, heads, dim, vdim, reinterpret_cast<float4*>(gates), q_scale, skip, state, norm_state,
                  slots, positions, seq_start, out, den, 0};
+  if (seq_start && !simple && chunks_fit(dtype, dim, vdim, max_q)) {
+    B200_REQUIRE(kind != B200F_MEMORY_DELTA || (ws && aligned16(ws)), B200_E_NULL, "memory_scan: no workspace");
+    const bf16* r = (const bf16*)rows;
+    switch (kind) {
+      case B200F_MEMORY_EXP: return launch_chunks<B200F_MEMORY_EXP>(p, r, nullptr, tokens, batch, max_q, (cudaStream_t)s);
+      case B200F_MEMORY_SSD: return launch_chunks<B200F_MEMORY_SSD>(p, r, nullptr, tokens, batch, max_q, (cudaStream_t)s);
+      default: return launch_chunks<B200F_MEMORY_DELTA>(p, r, (bf16*)ws, tokens, batch, max_q, (cudaStream_t)s);
+    }
+  }
   return dtype == B200F_BF16 ? launch_memory(p, kind, (const bf16*)rows, batch, (cudaStream_t)s)
                              : launch_memory(p, kind, (const float*)rows, batch, (cudaStream_t)s);
+}
+
+extern "C" int b200f_memory_scan_status(int* out_host, int reset) {
+  B200_REQUIRE(out_host, B200_E_NULL, "memory_scan_status: null pointer");
+  cudaError_t e = cudaMemcpyFromSymbol(out_host, g_gemm_status, sizeof(int));
+  if (e == cudaSuccess && reset) {
+    const int zero = 0;
+    e = cudaMemcpyToSymbol(g_gemm_status, &zero, sizeof(int));
+  }
+  B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan_status: %s", cudaGetErrorString(e));
+  return B200_OK;
 }
 
 extern "C" int b200f_memory_output(const float* o, const float* den, int heads, int vdim, int group, const float* y, int splits,

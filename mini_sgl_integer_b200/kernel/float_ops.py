@@ -103,14 +103,15 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def check_status() -> None:
-    """Raises if a bounded wait inside a linear or the attention kernel has expired since the last check.  Synchronises
-    with the device."""
-    for name, what in (("b200f_gemm_status", "a bf16 linear"), ("b200f_latent_attn_status", "the latent attention kernel")):
+    """Raises if a bounded wait inside a linear, the latent attention kernel or the chunked scan has expired since the last
+    check.  Synchronises with the device."""
+    for name, what in (("b200f_gemm_status", "a bf16 linear"), ("b200f_latent_attn_status", "the latent attention kernel"),
+                       ("b200f_memory_scan_status", "the scan of a matrix memory")):
         st = ctypes.c_int(0)
         call(name, ctypes.byref(st), 1)
         if st.value:
             raise RuntimeError(f"a wait inside {what} expired (code {st.value}: 1 loader, 2 MMA issuer, 3 epilogue, 4 accumulator "
-                               "hand-back, 5 copying warp, 6 consumer); the step's results are not valid")
+                               "hand-back, 5 copying warp, 6 consumer, 7 chunk); the step's results are not valid")
 
 
 # ----------------------------------------------------------------------------- ends of a model
@@ -263,9 +264,10 @@ def memory_prepare(y: torch.Tensor, col0: int, segments, conv_w: Optional[torch.
 
 def memory_scan(rows_: torch.Tensor, offsets, qk_heads: int, heads: int, dim: int, vdim: int, kind: int, gates: torch.Tensor, q_scale: float,
                 skip: Optional[torch.Tensor], state: torch.Tensor, norm_state: Optional[torch.Tensor], slots, positions, seq_start,
-                out: torch.Tensor, den: Optional[torch.Tensor]) -> None:
+                out: torch.Tensor, den: Optional[torch.Tensor], max_q: int, simple: bool = False) -> None:
     """Read-outs of a matrix recurrence; ``state`` fp32 [slots, heads, dim, round8(vdim)] is updated; see b200f_memory_scan.
-    ``offsets``: columns of the first q, k and v head; out fp32 [T, heads * vdim], den fp32 [T, heads]."""
+    ``offsets``: columns of the first q, k and v head; out fp32 [T, heads * vdim], den fp32 [T, heads].  ``max_q``: most new
+    tokens of a sequence; ``simple``: token by token also where chunks on the tensor cores would do."""
     T = rows_.shape[0]
     _check_rows("rows", rows_, rows_.dtype)
     _check_vec("gates", gates, T * heads * 4)
@@ -278,8 +280,11 @@ def memory_scan(rows_: torch.Tensor, offsets, qk_heads: int, heads: int, dim: in
         _check_vec("den", den, T * heads)
         if norm_state.shape[1:] != (heads, dim + 1) or not norm_state.is_contiguous():
             raise ValueError(f"norm_state must be contiguous fp32 [slots, {heads}, {dim + 1}]")
+    need = 0 if simple or seq_start is None else query("b200f_memory_scan_ws_bytes", T, slots.numel(), max_q, heads, dim, vdim, kind, dtype_code(rows_.dtype))
+    ws = torch.empty(need, dtype=torch.uint8, device=rows_.device) if need else None
     call("b200f_memory_scan", ptr(rows_), dtype_code(rows_.dtype), _pitch(rows_), *offsets, qk_heads, heads, dim, vdim, kind, ptr(gates),
-         float(q_scale), ptr(skip), ptr(state), ptr(norm_state), ptr(slots), ptr(positions), ptr(seq_start), ptr(out), ptr(den), T, slots.numel(), stream())
+         float(q_scale), ptr(skip), ptr(state), ptr(norm_state), ptr(slots), ptr(positions), ptr(seq_start), ptr(out), ptr(den), T, slots.numel(),
+         max_q, ptr(ws), int(simple), stream())
 
 
 def memory_output(o: torch.Tensor, den: Optional[torch.Tensor], heads: int, vdim: int, group: int, y: torch.Tensor, gate_col: int, gate: int,

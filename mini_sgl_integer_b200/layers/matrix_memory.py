@@ -53,7 +53,8 @@ class MatrixMemory(BaseOP):
                           md.positions, md.seq_start, md.seq_ids, rows, self.kind, H, [col + c for c in self._gate_cols], self.gate_a, self.gate_b,
                           gates, self._cap, n)
         fo.memory_scan(rows, self._offsets, self._qk, H, self._dim, self._vdim, self.kind, gates, self._q_scale, self._skip,
-                       cache.state(index, "S"), n, md.slots, md.positions, md.seq_start, o, den)
+                       cache.state(index, "S"), n, md.slots, md.positions, md.seq_start, o, den,
+                       md.max_seqlen_q)
         out = fo.rows(T, H * self._vdim, dtype, dev)
         fo.memory_output(o, den, H, self._vdim, self._group, y, col + self._out_gate, self.gate, self.norm, self._eps, out)
         return self.o.parts(out)

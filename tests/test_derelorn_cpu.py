@@ -78,7 +78,7 @@ def test_entry_points_reject_bad_arguments_before_launch():
     assert code(*prepare(ok, start=one)) == -1                     # sequence bounds without sequence ids
     assert code(*prepare(ok, kind=0)) == -2                        # exponential gates without their state
     scan = lambda dim=8, heads=2, qk=2, q_off=0, pitch=48, den=None, kind=1, dtype=1: (
-        "b200f_memory_scan", one, dtype, pitch, q_off, 16, 32, qk, heads, dim, 8, kind, one, 1.0, None, one, None, one, one, None, one, den, 3, 3, None)
+        "b200f_memory_scan", one, dtype, pitch, q_off, 16, 32, qk, heads, dim, 8, kind, one, 1.0, None, one, None, one, one, None, one, den, 3, 3, 1, None, 0, None)
     assert code(*scan(qk=3)) == -2
     assert code(*scan(pitch=40)) == -2
     assert code(*scan(dim=600)) == -4
