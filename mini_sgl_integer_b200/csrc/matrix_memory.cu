@@ -548,7 +548,7 @@ __device__ __forceinline__ int64_t chunk_index(int64_t first_token, int seq, int
 
 __host__ __device__ constexpr int chunk_panels(int dr) { return dr <= 4 ? 1 : dr / 4; }
 __host__ __device__ constexpr size_t chunk_smem(int dr, bool delta) {
-  return (size_t)(2 * chunk_panels(dr) + (delta ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 8 + 1024;
+  return (size_t)(2 * chunk_panels(dr) + (delta ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 2 * kChunk * 16 + 8 + 1024;
 }
 // Byte offset of (row, col) in a panel.
 __host__ __device__ __forceinline__ int panel_at(int row, int col) { return row * 128 + ((((col >> 3) ^ row) & 7) << 4) + (col & 7) * 2; }
@@ -563,7 +563,7 @@ __device__ __forceinline__ void sum64(float& a, float& b, int lane) {
   b += __shfl_sync(FULL_MASK, a, 31);
 }
 
-template <int KIND, int DR>
+template <int KIND, int DR, bool FULL>      // FULL: dim is exactly 16 DR
 __global__ void __launch_bounds__(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0), DR > 8 ? 1 : (DR == 8 && KIND == B200F_MEMORY_EXP ? 2 : 3))
 memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams p, const bf16* __restrict__ inverse) {
   extern __shared__ __align__(16) unsigned char smem[];
@@ -581,7 +581,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
   const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, col0 = slice * kChunkCols;
   const int vp = p.vdim, k16 = p.dim >> 4, qh = h / (p.heads / p.qk_heads);
-  const unsigned bar = smem_u32(es + C);
+  float4* gs = reinterpret_cast<float4*>(es + C);        // [2][C]
+  const unsigned bar = smem_u32(gs + 2 * C);
   if (tid == 0) {
     mbar_init(bar, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -610,7 +611,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     for (int k = 0; k < 4; ++k) {
       const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
       float v = 0.0f;
-      if (has_state && works && d < p.dim) {
+      if (has_state && works && (FULL || d < p.dim)) {
         if (is_n) v = k < 2 && g == 0 ? nst[d] : 0.0f;
         else if (col0 + c < vp) v = st[(int64_t)d * vp + c];
       }
@@ -620,14 +621,23 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
   // ldmatrix addresses: rows of 128 bytes, 16-byte pieces exchanged by the row's last three bits
   const unsigned n_row = ((lane & 7) + ((lane >> 4) << 3)) * 128, n_x = (((lane >> 3) & 1) ^ (lane & 7)) << 4;     // right operand from [n][k], left from [k][m]
   const unsigned m_row = (lane & 15) * 128, m_x = ((lane >> 4) ^ (lane & 7)) << 4;                                 // left operand from [m][k], right from [k][n]
-  auto at_n = [&](unsigned base, int row16, int k16th) { return base + (k16th >> 2) * kPanel + row16 * 2048 + n_row + (n_x ^ ((k16th & 3) << 5)); };
-  auto at_m = [&](unsigned base, int row16, int k16th) { return base + (k16th >> 2) * kPanel + row16 * 2048 + m_row + (m_x ^ ((k16th & 3) << 5)); };
+  unsigned n_at[4], m_at[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    n_at[i] = q_base + n_row + (n_x ^ (i << 5));
+    m_at[i] = q_base + m_row + (m_x ^ (i << 5));
+  }
+  // `panel`: number of a panel from q's first on
+  auto at_n = [&](int panel, int row16, int k16th) { return n_at[k16th & 3] + (panel + (k16th >> 2)) * kPanel + row16 * 2048; };
+  auto at_m = [&](int panel, int row16, int k16th) { return m_at[k16th & 3] + (panel + (k16th >> 2)) * kPanel + row16 * 2048; };
+  constexpr int Q_ = 0, K_ = DP, V_ = 2 * DP, PL_ = V_ + 1, PH_ = DELTA ? V_ : PL_ + 1, T_ = PL_ + 1;
+  const unsigned v_at = q_base + V_ * kPanel + n_row + (n_x ^ ((warp & 3) << 5));
 
   // acc [16 columns, 64 tokens] = S^T X^T for X = q or k
-  auto state_times = [&](unsigned x_base, float (&acc)[8][4]) {
+  auto state_times = [&](int x, float (&acc)[8][4]) {
 #pragma unroll
     for (int kk = 0; kk < DR; ++kk) {
-      if (kk >= k16) break;
+      if (!FULL && kk >= k16) break;
       unsigned ah[4], al[4];
       split2(S[2 * kk][0], S[2 * kk][1], &ah[0], &al[0]);
       split2(S[2 * kk][2], S[2 * kk][3], &ah[1], &al[1]);
@@ -635,7 +645,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       split2(S[2 * kk + 1][2], S[2 * kk + 1][3], &ah[3], &al[3]);
       unsigned b[4][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) mm_ldsm(b[j], at_n(x_base, j, kk));
+      for (int j = 0; j < 4; ++j) mm_ldsm(b[j], at_n(x, j, kk));
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         mm_mma(acc[2 * j], ah, b[j][0], b[j][1]);
@@ -654,17 +664,18 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       a[0] = a[2] = g == 0 ? 0x3f803f80u : 0u;           // ones
       a[1] = a[3] = 0u;
     } else {
-      mm_ldsm_t(a, at_n(v_base, kb, warp));
+      mm_ldsm_t(a, v_at + kb * 2048);
     }
   };
 
   const int chunks = (count + C - 1) / C;
-  float4 gate_a, gate_b;                                  // warp 0: the next chunk's gates
-  auto load_gates = [&](int ch) {
-    const float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    const float4* src = p.gates + (t0 + (int64_t)ch * C + lane) * p.heads + h;
-    gate_a = ch * C + lane < count ? src[0] : z;
-    gate_b = ch * C + lane + 32 < count ? src[(int64_t)32 * p.heads] : z;
+  auto load_gates = [&](int ch) {                         // by warp 0, a chunk ahead; entries behind the portion are not used
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = lane + 32 * half;
+      if (ch * C + t < count) cp_async16(smem_u32(gs + (ch & 1) * C + t), p.gates + (t0 + (int64_t)ch * C + t) * p.heads + h);
+    }
+    cp_async_commit();
   };
   if (warp == 0) load_gates(0);
   for (int ch = 0; ch < chunks; ++ch) {
@@ -682,8 +693,11 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         if (DELTA) bulk_copy(t_base, inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C), 2 * kPanel, bar);
       }
       __syncwarp();
-      const float4 ga = gate_a, gb = gate_b;
       load_gates(ch + 1);
+      cp_async_wait<1>();
+      __syncwarp();
+      const float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f), *src = gs + (ch & 1) * C;
+      const float4 ga = lane < n ? src[lane] : z, gb = lane + 32 < n ? src[lane + 32] : z;
       float la = ga.x * 1.4426950408889634f, lb = gb.x * 1.4426950408889634f;
       sum64(la, lb, lane);
       const float last = __shfl_sync(FULL_MASK, lb, 31);
@@ -710,7 +724,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     if (DELTA) {
       if (works) {
         float r[8][4] = {};                               // right-hand side beta (v - e^L K S_0), transposed
-        state_times(k_base, r);
+        state_times(K_, r);
 #pragma unroll
         for (int kb = 0; kb < 4; ++kb) {
           unsigned v[4];
@@ -740,8 +754,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
           unsigned bh[4][4], bl[4][4];
 #pragma unroll
           for (int j = kb; j < 4; ++j) {
-            mm_ldsm(bh[j], at_n(t_base, j, kb));
-            mm_ldsm(bl[j], at_n(t_base + kPanel, j, kb));
+            mm_ldsm(bh[j], at_n(T_, j, kb));
+            mm_ldsm(bl[j], at_n(T_ + 1, j, kb));
           }
 #pragma unroll
           for (int j = kb; j < 4; ++j) {
@@ -772,13 +786,13 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       for (int k = 0; k < 8; ++k) sc[m][k >> 2][k & 3] = 0.0f;
 #pragma unroll
     for (int kk = 0; kk < DR; ++kk) {
-      if (kk >= k16) break;
+      if (!FULL && kk >= k16) break;
       unsigned a[MINE][4], b[MINE][4];
 #pragma unroll
       for (int m = 0; m < MINE; ++m) {
         const int blk = min(warp + m * WARPS, 9), rb = (blk >= 1) + (blk >= 3) + (blk >= 6), kb = blk - rb * (rb + 1) / 2;
-        mm_ldsm(a[m], at_m(q_base, rb, kk));
-        mm_ldsm(b[m], at_n(k_base, kb, kk));
+        mm_ldsm(a[m], at_m(Q_, rb, kk));
+        mm_ldsm(b[m], at_n(K_, kb, kk));
       }
 #pragma unroll
       for (int m = 0; m < MINE; ++m) {
@@ -819,7 +833,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
 
     if (works) {
       float o[8][4] = {};
-      state_times(q_base, o);
+      state_times(Q_, o);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const float2 e = *reinterpret_cast<const float2*>(el + i * 8 + q2);
@@ -859,8 +873,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         unsigned bh[4][4], bl[4][4];
 #pragma unroll
         for (int j = kb; j < 4; ++j) {
-          mm_ldsm(bh[j], at_n(ph_base, j, kb));
-          mm_ldsm(bl[j], at_n(pl_base, j, kb));
+          mm_ldsm(bh[j], at_n(PH_, j, kb));
+          mm_ldsm(bl[j], at_n(PL_, j, kb));
         }
 #pragma unroll
         for (int j = kb; j < 4; ++j) {
@@ -882,10 +896,10 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         constexpr int KG = DR < 4 ? DR : 4;
 #pragma unroll
         for (int k0 = 0; k0 < DR; k0 += KG) {
-          if (k0 >= k16) break;
+          if (!FULL && k0 >= k16) break;
           unsigned b[KG][4];
 #pragma unroll
-          for (int i = 0; i < KG; ++i) mm_ldsm_t(b[i], at_m(k_base, kb, k0 + i));
+          for (int i = 0; i < KG; ++i) mm_ldsm_t(b[i], at_m(K_, kb, k0 + i));
 #pragma unroll
           for (int i = 0; i < KG; ++i) {
             mm_mma(S[2 * (k0 + i)], dh, b[i][0], b[i][1]);
@@ -933,7 +947,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
-      if (d >= p.dim) continue;
+      if (!FULL && d >= p.dim) continue;
       if (is_n) {
         if (k < 2 && g == 0) nst[d] = S[i][k];
       } else if (col0 + c < vp) {
@@ -1276,14 +1290,14 @@ static int launch_scan_shape(MemoryParams p, const T* rows, int batch, cudaStrea
   launch_pdl(memory_scan_kernel<T, KIND, LN, R>, grid, dim3(32 * warps + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, p, rows);
   return check_launch("memory_scan");
 }
-template <int KIND, int DR>
+template <int KIND, int DR, bool FULL>
 static int launch_chunk_shape(const CUtensorMap& map, const MemoryParams& p, const bf16* inverse, int batch, cudaStream_t st) {
   constexpr size_t bytes = chunk_smem(DR, KIND == B200F_MEMORY_DELTA);
   static_assert(bytes <= 227 * 1024, "shared memory budget");
-  cudaError_t e = cudaFuncSetAttribute(memory_chunk_kernel<KIND, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+  cudaError_t e = cudaFuncSetAttribute(memory_chunk_kernel<KIND, DR, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
   B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
   const dim3 grid((unsigned)((p.vdim + kChunkCols - 1) / kChunkCols), (unsigned)p.heads, (unsigned)batch);
-  launch_pdl(memory_chunk_kernel<KIND, DR>, grid, dim3(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, map, p, inverse);
+  launch_pdl(memory_chunk_kernel<KIND, DR, FULL>, grid, dim3(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, map, p, inverse);
   return check_launch("memory_scan (chunks)");
 }
 template <int KIND>
@@ -1306,10 +1320,13 @@ static int launch_chunks(const MemoryParams& p, const bf16* rows, bf16* inverse,
     const int rc = check_launch("memory_scan (inverse)");
     if (rc != B200_OK) return rc;
   }
-  if (p.dim <= 32) return launch_chunk_shape<KIND, 2>(map, p, inverse, batch, st);
-  if (p.dim <= 64) return launch_chunk_shape<KIND, 4>(map, p, inverse, batch, st);
-  if (p.dim <= 128) return launch_chunk_shape<KIND, 8>(map, p, inverse, batch, st);
-  return launch_chunk_shape<KIND, 16>(map, p, inverse, batch, st);
+  if (p.dim == 32) return launch_chunk_shape<KIND, 2, true>(map, p, inverse, batch, st);
+  if (p.dim < 32) return launch_chunk_shape<KIND, 2, false>(map, p, inverse, batch, st);
+  if (p.dim == 64) return launch_chunk_shape<KIND, 4, true>(map, p, inverse, batch, st);
+  if (p.dim < 64) return launch_chunk_shape<KIND, 4, false>(map, p, inverse, batch, st);
+  if (p.dim == 128) return launch_chunk_shape<KIND, 8, true>(map, p, inverse, batch, st);
+  if (p.dim < 128) return launch_chunk_shape<KIND, 8, false>(map, p, inverse, batch, st);
+  return p.dim == 256 ? launch_chunk_shape<KIND, 16, true>(map, p, inverse, batch, st) : launch_chunk_shape<KIND, 16, false>(map, p, inverse, batch, st);
 }
 // The chunk form: bf16 heads of whole 16-value pieces (q, k) and without padding (v), and portions that fill a good part of a chunk.
 static bool chunks_fit(int dtype, int dim, int vdim, int max_q) { return dtype == B200F_BF16 && dim <= 256 && dim % 16 == 0 && vdim % 8 == 0 && max_q > 16; }
