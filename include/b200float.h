@@ -128,7 +128,8 @@ B200_API int b200f_latent_attn_status(int* out_host, int reset);   /* as b200f_g
  * b200f_memory_scan_ws_bytes bytes.  The other two entries of a token's gates may be overwritten.
  *
  * b200f_memory_output: u = o / den (den nullable); groups of `group` values of a row are divided by their root mean square
- * (eps inside) and multiplied by norm_w[column % norm_len]; the gate is the projection in column gate_col of y: silu(gate)
+ * (eps inside) and multiplied by norm_w (a gain per column, or norm_len == group gains for every group; with den, a group is
+ * a head); the gate is the projection in column gate_col of y: silu(gate)
  * in front of the norm, or sigmoid(gate) or silu(gate) behind it. */
 enum { B200F_MEMORY_EXP = 0, B200F_MEMORY_SSD = 1, B200F_MEMORY_DELTA = 2 };
 enum { B200F_GATE_SILU_BEFORE = 0, B200F_GATE_SIGMOID_AFTER = 1, B200F_GATE_SILU_AFTER = 2 };

@@ -159,9 +159,9 @@ __device__ __forceinline__ void ga_ldsm_t(unsigned (&r)[4], unsigned addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 __device__ __forceinline__ void ga_mma(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ float ga_exp2(float v) {
   float r;
@@ -171,15 +171,16 @@ __device__ __forceinline__ float ga_exp2(float v) {
 
 __host__ __device__ constexpr int ga_ld(int n) { return ((n + 15) & ~15) + 8; }         // shared row pitch: conflict-free ldmatrix
 
-// D16: most 16-column pieces of a key or value.  DECODE: every warp has the same 16 rows and a quarter of each key tile.
-template <int D16, bool DECODE>
+// D16: most 16-column pieces of a key or value; FULL: exactly that many.  DECODE: every warp has the same 16 rows and a quarter
+// of each key tile.
+template <int D16, bool DECODE, bool FULL>
 __global__ void __launch_bounds__(kGaWarps * 32)
 grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, const bf16* __restrict__ k_cache,
                         const bf16* __restrict__ v_cache, bf16* __restrict__ out) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   constexpr int NT = kGaTile, THREADS = kGaWarps * 32;
   constexpr int KW = DECODE ? NT / kGaWarps : NT;                      // keys of a tile per warp
-  const int ldk = ga_ld(p.dim), ldv = ga_ld(p.vdim);
+  const int ldk = FULL ? ga_ld(16 * D16) : ga_ld(p.dim), ldv = FULL ? ga_ld(16 * D16) : ga_ld(p.vdim);
   const int k16 = (p.dim + 15) >> 4, c16 = (p.vdim + 15) >> 4;
   bf16* ks = reinterpret_cast<bf16*>(smem_raw);                        // [2][NT][ldk]
   bf16* vs = ks + 2 * NT * ldk;                                        // [2][NT][ldv]
@@ -207,19 +208,43 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
   const int tile0 = split * per_split, tile1 = min(all_tiles, tile0 + per_split);
   const int32_t* pages = p.page_table + (int64_t)seq * p.table_pitch;
 
-  // a row is copied by as many threads as it has 16-byte pieces; keys outside [key_lo, key_hi) repeat a visible one
-  const int ck = p.dim_pitch / 8, cv = p.vdim_pitch / 8, chunks = ck + cv;
-  auto issue = [&](int tile) {
-    const int buf = (tile - tile0) & 1, k0 = base + tile * NT;
-    for (int i = threadIdx.x; i < NT * chunks; i += THREADS) {
-      const int r = i / chunks, c = i - r * chunks;
-      const int key = min(max(k0 + r, key_lo), key_hi - 1);
-      const int64_t row = ((int64_t)__ldg(pages + key / kGaPage) * kGaPage + key % kGaPage) * p.kv_heads + kvh;
-      if (c < ck) cp_async16(smem_u32(ks + (buf * NT + r) * ldk + c * 8), k_cache + row * p.dim_pitch + c * 8);
-      else cp_async16(smem_u32(vs + (buf * NT + r) * ldv + (c - ck) * 8), v_cache + row * p.vdim_pitch + (c - ck) * 8);
+  // Each warp copies one of a tile's four pages, a 16-byte piece of the key or value of all 16 rows per lane; keys outside
+  // [key_lo, key_hi) become zeros.  The page id is looked up a tile ahead.
+  static_assert(NT == kGaWarps * kGaPage, "a page per warp");
+  const int ck = p.dim_pitch / 8, chunks = ck + p.vdim_pitch / 8, last_page = (key_hi - 1) / kGaPage;
+  int page = 0;
+  auto look_up = [&](int tile) { page = __ldg(pages + min((base + tile * NT) / kGaPage + warp, last_page)); };
+  auto issue = [&](int tile) {                   // needs look_up(tile)
+    const int buf = (tile - tile0) & 1, r0 = warp * kGaPage, k0 = base + tile * NT + r0;
+    const bool all = k0 >= key_lo && k0 + kGaPage <= key_hi;
+    for (int c = lane; c < chunks; c += 32) {
+      const bool is_k = c < ck;
+      const int pitch = is_k ? p.dim_pitch : p.vdim_pitch, col = (is_k ? c : c - ck) * 8, ld = is_k ? ldk : ldv;
+      const bf16* src = (is_k ? k_cache : v_cache) + ((int64_t)page * kGaPage * p.kv_heads + kvh) * pitch + col;
+      unsigned dst = smem_u32((is_k ? ks : vs) + (buf * NT + r0) * ld + col);
+      const int64_t step = (int64_t)p.kv_heads * pitch;
+      if (all) {
+#pragma unroll
+        for (int r = 0; r < kGaPage; ++r) {
+          cp_async16(dst, src);
+          src += step;
+          dst += 2 * ld;
+        }
+      } else {
+        for (int r = 0; r < kGaPage; ++r) {
+          const int live = k0 + r >= key_lo && k0 + r < key_hi ? 16 : 0;
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live) : "memory");
+          src += step;
+          dst += 2 * ld;
+        }
+      }
     }
+    if (tile + 1 < tile1) look_up(tile + 1);
   };
-  if (tile0 < tile1) issue(tile0);
+  if (tile0 < tile1) {
+    look_up(tile0);
+    issue(tile0);
+  }
   cp_async_commit();
 
   const int row_base = DECODE ? 0 : warp * 16;
@@ -260,6 +285,9 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
   const int warp_lo = DECODE ? key_lo : ga_first_key(pos0 + min(row_base, rows - 1) / nh, p.window);
   const int warp_hi = DECODE ? key_hi : pos0 + min(row_base + 15, rows - 1) / nh + 1;
   const bool warp_live = row_base < rows;
+  // keys [all_lo, all_hi) are seen by every row (rows behind the last one do not matter)
+  const int all_lo = ga_first_key(pos0 + (DECODE ? ntok - 1 : min(row_base + 15, rows - 1) / nh), p.window);
+  const int all_hi = pos0 + (DECODE ? 0 : min(row_base, rows - 1) / nh) + 1;
 
   for (int tile = tile0; tile < tile1; ++tile) {
     const int buf = (tile - tile0) & 1;
@@ -277,7 +305,7 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
       const unsigned kb = smem_u32(ks + buf * NT * ldk + k_lane);
 #pragma unroll
       for (int i = 0; i < D16; ++i) {
-        if (i < k16) {
+        if (FULL || i < k16) {
 #pragma unroll
           for (int n = 0; n < KW / 16; ++n) {
             unsigned b[4];
@@ -288,14 +316,24 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
         }
       }
       float mn[2] = {m[0], m[1]};
+      if (key0 >= all_lo && key0 + KW <= all_hi) {
 #pragma unroll
-      for (int i = 0; i < KW / 8; ++i)
+        for (int i = 0; i < KW / 8; ++i)
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int key = key0 + 8 * i + 2 * (lane & 3) + (k & 1), r = k >> 1;
-          s[i][k] = (key <= vis_hi[r] && key >= vis_lo[r]) ? s[i][k] * p.scale2 : -INFINITY;
-          mn[r] = fmaxf(mn[r], s[i][k]);
-        }
+          for (int k = 0; k < 4; ++k) {
+            s[i][k] *= p.scale2;
+            mn[k >> 1] = fmaxf(mn[k >> 1], s[i][k]);
+          }
+      } else {
+#pragma unroll
+        for (int i = 0; i < KW / 8; ++i)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int key = key0 + 8 * i + 2 * (lane & 3) + (k & 1), r = k >> 1;
+            s[i][k] = (key <= vis_hi[r] && key >= vis_lo[r]) ? s[i][k] * p.scale2 : -INFINITY;
+            mn[r] = fmaxf(mn[r], s[i][k]);
+          }
+      }
       float alpha[2], mu[2];
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
@@ -329,7 +367,7 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
                                f32_to_bf16x2(s[2 * kk + 1][0], s[2 * kk + 1][1]), f32_to_bf16x2(s[2 * kk + 1][2], s[2 * kk + 1][3])};
 #pragma unroll
         for (int i = 0; i < D16; ++i) {
-          if (i < c16) {
+          if (FULL || i < c16) {
             unsigned b[4];
             ga_ldsm_t(b, vb + (unsigned)(kk * 16 * ldv * 2) + 32 * i);
             ga_mma(acc[i][0], a, b[0], b[1]);
@@ -408,7 +446,7 @@ grouped_attn_mma_kernel(const GroupedAttn p, const bf16* __restrict__ q_in, cons
     const bool pair = ((reinterpret_cast<uintptr_t>(dst) & 3) == 0);
 #pragma unroll
     for (int i = 0; i < D16; ++i)
-      if (i < c16) {
+      if (FULL || i < c16) {
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           const int col = i * 16 + 8 * j + 2 * (lane & 3);
@@ -456,11 +494,11 @@ static size_t ga_smem(int dim, int vdim, bool decode) {
 static bool ga_decode_form(int max_q, int heads, int kv_heads) { return max_q == 1 && heads / kv_heads > 0; }
 static int ga_rows(bool decode) { return decode ? 16 : 16 * kGaWarps; }
 
-template <int D16, bool DECODE>
+template <int D16, bool DECODE, bool FULL>
 static int launch_ga(const GroupedAttn& p, const bf16* q, const bf16* k, const bf16* v, bf16* out, dim3 grid, size_t smem, cudaStream_t st) {
-  cudaError_t e = cudaFuncSetAttribute(grouped_attn_mma_kernel<D16, DECODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(grouped_attn_mma_kernel<D16, DECODE, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "grouped_attn: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
-  launch_pdl(grouped_attn_mma_kernel<D16, DECODE>, grid, dim3(kGaWarps * 32), smem, st, p, q, k, v, out);
+  launch_pdl(grouped_attn_mma_kernel<D16, DECODE, FULL>, grid, dim3(kGaWarps * 32), smem, st, p, q, k, v, out);
   return check_launch("grouped_attn");
 }
 static bool ga_mma_fits(int dim, int vdim, int dtype) {
@@ -550,10 +588,15 @@ extern "C" int b200f_grouped_attn(const void* q, const void* k_cache, const void
   bf16* o = (bf16*)out;
   const int big = dim > vdim ? dim : vdim;
   int rc;
-  if (decode) rc = big <= 64 ? launch_ga<4, true>(p, qq, kk, vv, o, grid, smem, st)
-                             : (big <= 128 ? launch_ga<8, true>(p, qq, kk, vv, o, grid, smem, st) : launch_ga<16, true>(p, qq, kk, vv, o, grid, smem, st));
-  else rc = big <= 64 ? launch_ga<4, false>(p, qq, kk, vv, o, grid, smem, st)
-                      : (big <= 128 ? launch_ga<8, false>(p, qq, kk, vv, o, grid, smem, st) : launch_ga<16, false>(p, qq, kk, vv, o, grid, smem, st));
+#define B200_GA_CASE(D16_)                                                                                                                     \
+  if (dim == 16 * D16_ && vdim == dim)                                                                                                        \
+    rc = decode ? launch_ga<D16_, true, true>(p, qq, kk, vv, o, grid, smem, st) : launch_ga<D16_, false, true>(p, qq, kk, vv, o, grid, smem, st);   \
+  else                                                                                                                                        \
+    rc = decode ? launch_ga<D16_, true, false>(p, qq, kk, vv, o, grid, smem, st) : launch_ga<D16_, false, false>(p, qq, kk, vv, o, grid, smem, st);
+  if (big <= 64) { B200_GA_CASE(4) }
+  else if (big <= 128) { B200_GA_CASE(8) }
+  else { B200_GA_CASE(16) }
+#undef B200_GA_CASE
   if (rc != B200_OK || key_splits == 1) return rc;
   launch_pdl(grouped_merge_kernel, dim3((unsigned)(tokens * heads)), dim3(128), 0, st, p, o);
   return check_launch("grouped_attn (merge)");

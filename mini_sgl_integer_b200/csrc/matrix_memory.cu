@@ -459,7 +459,6 @@ memory_scan_kernel(const MemoryParams p, const T* __restrict__ rows) {
 // Log gates (f, i) of a prompt batch to (f + m_(t-1) - m_t, exp(i - m_t), exp(-m_t)); a warp per (sequence, head).
 __global__ void __launch_bounds__(32)
 running_max_kernel(const MemoryPrepare p) {
-  __shared__ float2 fi[32];
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.x, seq = blockIdx.y, lane = threadIdx.x;
@@ -467,22 +466,27 @@ running_max_kernel(const MemoryPrepare p) {
   if (t0 >= t1) return;
   float* ms = p.norm_state + ((int64_t)p.slots[seq] * p.heads + h) * (p.norm_dim + 1) + p.norm_dim;
   float m = p.positions[t0] > 0 ? *ms : 0.0f;
-  float4 next = t0 + lane < t1 ? p.gates[(t0 + lane) * p.heads + h] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  const float4 none = make_float4(0.0f, -INFINITY, 0.0f, 0.0f);         // leaves the maximum alone
+  auto load = [&](int64_t t) { return t < t1 ? p.gates[t * p.heads + h] : none; };
+  float4 next[2] = {load(t0 + lane), load(t0 + 32 + lane)};
   for (int64_t base = t0; base < t1; base += 32) {
-    const int n = (int)min((int64_t)32, t1 - base);
-    const float4 g = next;
-    __syncwarp();
-    fi[lane] = make_float2(g.x, g.y);
-    __syncwarp();
-    if (base + 32 + lane < t1) next = p.gates[(base + 32 + lane) * p.heads + h];
-    float before = m, after = m;
-    for (int t = 0; t < n; ++t) {
-      const float2 u = fi[t];
-      const float nm = fmaxf(u.x + m, u.y);
-      if (t == lane) { before = m; after = nm; }
-      m = nm;
+    const float4 g = next[0];
+    next[0] = next[1];
+    next[1] = load(base + 64 + lane);
+    float a = g.x, b = g.y;                              // m -> max(m + a, b), composed over the lanes up to this one
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pa = __shfl_up_sync(FULL_MASK, a, o), pb = __shfl_up_sync(FULL_MASK, b, o);
+      if (lane >= o) {
+        b = fmaxf(pb + a, b);
+        a += pa;
+      }
     }
-    if (lane < n) p.gates[(base + lane) * p.heads + h] = make_float4(g.x + before - after, expf(g.y - after), expf(-after), 0.0f);
+    const float after = fmaxf(m + a, b);
+    float before = __shfl_up_sync(FULL_MASK, after, 1);
+    if (lane == 0) before = m;
+    m = __shfl_sync(FULL_MASK, after, 31);
+    if (base + lane < t1) p.gates[(base + lane) * p.heads + h] = make_float4(fminf(g.x + before - after, 0.0f), expf(g.y - after), expf(-after), 0.0f);
   }
   if (lane == 0) *ms = m;
 }
@@ -987,15 +991,22 @@ delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* 
   cp_async_commit();
   for (int r = tid; r < C; r += 128)
     for (int c = p.dim; c < lk; ++c) ks[r * lk + c] = __float2bfloat16_rn(0.0f);
-  for (int t = warp; t < C; t += 4) {
+  {                                                      // two threads per token
+    const int t = tid >> 1;
+    const uint4* src = reinterpret_cast<const uint4*>(q_src + (int64_t)(t < n ? t : 0) * p.row_pitch + (tid & 1) * (p.dim / 2));
     float ss = 0.0f;
-    if (t < n)
-      for (int c = lane * 2; c < p.dim; c += 64) {
-        const float2 x = bf16x2_to_f32(*reinterpret_cast<const unsigned*>(q_src + (int64_t)t * p.row_pitch + c));
+#pragma unroll 4
+    for (int c = 0; c < p.dim / 16; ++c) {
+      const uint4 v = __ldg(src + c);
+      const unsigned w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 x = bf16x2_to_f32(w[k]);
         ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
       }
-    ss = warp_sum(ss);
-    if (lane == 0) rq[t] = p.q_scale / sqrtf(ss + kUnitEps);
+    }
+    ss += __shfl_xor_sync(FULL_MASK, ss, 1);
+    if ((tid & 1) == 0) rq[t] = p.q_scale / sqrtf(ss + kUnitEps);
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -1184,11 +1195,15 @@ struct MemoryOutput {
   int64_t out_pitch;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(256)
+// One CTA per row.  A warp per group, or several for the wide groups of a few; up to kOutKeep packs of a group per lane stay in
+// registers between the sum of squares and the result, the others are formed twice.
+constexpr int kOutKeep = 2;
+template <int V>
+struct alignas(4 * V) OutPack { float v[V]; };
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256, 4)
 memory_output_kernel(const MemoryOutput p, T* __restrict__ out) {
-  extern __shared__ __align__(16) unsigned char smem[];
-  float* u = reinterpret_cast<float*>(smem);          // [heads * vdim]
   __shared__ float part[8];
   pdl_launch_dependents();
   pdl_wait();
@@ -1198,20 +1213,50 @@ memory_output_kernel(const MemoryOutput p, T* __restrict__ out) {
   const float* o = p.o + row * n;
   const float* gate = p.y + row * p.y_pitch + p.gate_col;
   const int wpg = groups >= 8 ? 1 : 8 / groups, at_once = 8 / wpg, sub = warp % wpg;       // warps per group
+  const int step = 32 * wpg * V;
+  auto load = [&](const float* src) { return *reinterpret_cast<const OutPack<V>*>(src); };
+  auto gate_at = [&](int c) {
+    OutPack<V> z = load(gate + c);
+    for (int s = 1; s < p.splits; ++s) {
+      const OutPack<V> x = load(gate + c + s * p.split_stride);
+#pragma unroll
+      for (int k = 0; k < V; ++k) z.v[k] += x.v[k];
+    }
+    return z;
+  };
   for (int g0 = 0; g0 < groups; g0 += at_once) {
     const int g = g0 + warp / wpg;
     const bool live = warp / wpg < at_once && g < groups;
+    const int c0 = g * p.group;
+    const float inv_den = live && p.den ? 1.0f / p.den[row * p.heads + g] : 1.0f;         // with den a group is a head
+    auto value = [&](int i) {
+      OutPack<V> u = load(o + c0 + i);
+      if (p.gate == B200F_GATE_SILU_BEFORE) {
+        const OutPack<V> z = gate_at(c0 + i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) u.v[k] *= silu_f32(z.v[k]);
+      }
+      return u;
+    };
+    OutPack<V> keep[kOutKeep], z[kOutKeep];
     float ss = 0.0f;
-    if (live) {
-      for (int i = sub * 32 + lane; i < p.group; i += 32 * wpg) {
-        const int c = g * p.group + i;
-        float v = o[c];
-        if (p.den) v /= p.den[row * p.heads + c / p.vdim];
-        if (p.gate == B200F_GATE_SILU_BEFORE) v *= silu_f32(part_sum(gate + c, p.splits, p.split_stride));
-        u[c] = v;
-        ss = fmaf(v, v, ss);
+    const int first = (sub * 32 + lane) * V;
+#pragma unroll
+    for (int j = 0; j < kOutKeep; ++j) {
+      const int i = first + j * step;
+      if (live && i < p.group) {
+        keep[j] = value(i);
+        if (p.gate != B200F_GATE_SILU_BEFORE) z[j] = gate_at(c0 + i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) ss = fmaf(keep[j].v[k], keep[j].v[k], ss);
       }
     }
+    if (live)
+      for (int i = first + kOutKeep * step; i < p.group; i += step) {
+        const OutPack<V> u = value(i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) ss = fmaf(u.v[k], u.v[k], ss);
+      }
     ss = warp_sum(ss);
     if (wpg > 1) {
       if (lane == 0) part[warp] = ss;
@@ -1221,16 +1266,26 @@ memory_output_kernel(const MemoryOutput p, T* __restrict__ out) {
       __syncthreads();
     }
     if (!live) continue;
-    const float inv = 1.0f / sqrtf(ss / (float)p.group + p.eps);
-    for (int i = sub * 32 + lane; i < p.group; i += 32 * wpg) {
-      const int c = g * p.group + i;
-      float v = u[c] * inv * p.norm_w[c % p.norm_len];
-      if (p.gate != B200F_GATE_SILU_BEFORE) {
-        const float z = part_sum(gate + c, p.splits, p.split_stride);
-        v *= p.gate == B200F_GATE_SIGMOID_AFTER ? sigmoid_f32(z) : silu_f32(z);
+    const float inv = inv_den / sqrtf(ss * inv_den * inv_den / (float)p.group + p.eps);
+    const float* w = p.norm_w + (p.norm_len == n ? c0 : 0);
+    T* dst = out + row * p.out_pitch + c0;
+    auto finish = [&](int i, const OutPack<V>& u, const OutPack<V>& zz) {
+      const OutPack<V> gain = load(w + i);
+      OutPack<V> r;
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        r.v[k] = u.v[k] * inv * gain.v[k];
+        if (p.gate != B200F_GATE_SILU_BEFORE) r.v[k] *= p.gate == B200F_GATE_SIGMOID_AFTER ? sigmoid_f32(zz.v[k]) : silu_f32(zz.v[k]);
       }
-      out[row * p.out_pitch + c] = from_f32<T>(v);
-    }
+      if (V == 4) store4(dst + i, make_float4(r.v[0], r.v[V > 1 ? 1 : 0], r.v[V > 2 ? 2 : 0], r.v[V > 3 ? 3 : 0]));
+      else
+#pragma unroll
+        for (int k = 0; k < V; ++k) dst[i + k] = from_f32<T>(r.v[k]);
+    };
+#pragma unroll
+    for (int j = 0; j < kOutKeep; ++j)
+      if (first + j * step < p.group) finish(first + j * step, keep[j], z[j]);
+    for (int i = first + kOutKeep * step; i < p.group; i += step) finish(i, value(i), p.gate != B200F_GATE_SILU_BEFORE ? gate_at(c0 + i) : z[0]);
   }
 }
 
@@ -1459,15 +1514,24 @@ extern "C" int b200f_memory_output(const float* o, const float* den, int heads, 
   B200_REQUIRE(tokens >= 0 && tokens < (1ll << 31) && heads > 0 && vdim > 0 && group > 0 && n % group == 0 && norm_len > 0 && n % norm_len == 0 &&
                    splits >= 1 && gate_col >= 0 && gate_col + n <= y_pitch && out_pitch >= n, B200_E_SHAPE,
                "memory_output: tokens=%lld heads=%d vdim=%d group=%d", (long long)tokens, heads, vdim, group);
-  B200_REQUIRE(n * 4 <= 200 * 1024, B200_E_UNSUPPORTED, "memory_output: rows of %lld values are too wide", (long long)n);
+  B200_REQUIRE((norm_len == n || norm_len == group) && (!den || group == vdim), B200_E_UNSUPPORTED,
+               "memory_output: gains of %d for groups of %d, divisors per head of %d", norm_len, group, vdim);
   if (tokens == 0) return B200_OK;
   B200_REQUIRE(o && y && norm_w && out, B200_E_NULL, "memory_output: null pointer");
   MemoryOutput p{o, den, heads, vdim, group, y, splits, split_stride, y_pitch, gate_col, gate, norm_w, norm_len, eps, out_pitch};
-  const size_t bytes = (size_t)n * 4;
-  cudaError_t e = dtype == B200F_BF16 ? cudaFuncSetAttribute(memory_output_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes)
-                                      : cudaFuncSetAttribute(memory_output_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
-  B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_output: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
-  if (dtype == B200F_BF16) launch_pdl(memory_output_kernel<bf16>, dim3((unsigned)tokens), dim3(256), bytes, (cudaStream_t)s, p, (bf16*)out);
-  else launch_pdl(memory_output_kernel<float>, dim3((unsigned)tokens), dim3(256), bytes, (cudaStream_t)s, p, (float*)out);
+  const bool by4 = group % 4 == 0 && y_pitch % 4 == 0 && gate_col % 4 == 0 && split_stride % 4 == 0 && out_pitch % 4 == 0 && aligned16(o) && aligned16(y) &&
+                   aligned16(norm_w) && aligned16(out);
+  const int v = by4 && (group >= 128 || group % 2) ? 4 : (by4 && group >= 32 ? 2 : 1);      // narrow packs keep the lanes busy in small groups
+  const dim3 grid((unsigned)tokens), block(256);
+  cudaStream_t st = (cudaStream_t)s;
+  if (dtype == B200F_BF16) {
+    if (v == 4) launch_pdl(memory_output_kernel<bf16, 4>, grid, block, 0, st, p, (bf16*)out);
+    else if (v == 2) launch_pdl(memory_output_kernel<bf16, 2>, grid, block, 0, st, p, (bf16*)out);
+    else launch_pdl(memory_output_kernel<bf16, 1>, grid, block, 0, st, p, (bf16*)out);
+  } else {
+    if (v == 4) launch_pdl(memory_output_kernel<float, 4>, grid, block, 0, st, p, (float*)out);
+    else if (v == 2) launch_pdl(memory_output_kernel<float, 2>, grid, block, 0, st, p, (float*)out);
+    else launch_pdl(memory_output_kernel<float, 1>, grid, block, 0, st, p, (float*)out);
+  }
   return check_launch("memory_output");
 }
