@@ -986,6 +986,11 @@ def run_sefevik(args) -> None:
     bench_hybrid.run(args)
 
 
+def run_derelorn(args) -> None:
+    import bench_derelorn
+    bench_derelorn.run(args)
+
+
 def main() -> None:
     # NCCL only sets up the process group and runs the barriers / timing reductions around the step (the step itself
     # has no collective call), so it does not need in-switch reduction; the multi-GPU runs were validated with it off
@@ -995,7 +1000,7 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="model", choices=["model", "attn", "rowops", "gemm", "prefill", "offline", "tp_layer", "tp_linear", "sefevik"],
+    ap.add_argument("--workload", default="model", choices=["model", "attn", "rowops", "gemm", "prefill", "offline", "tp_layer", "tp_linear", "sefevik", "derelorn"],
                     help="model = the decode step of the 8B-shaped model, tensor-parallel over the launched ranks (default); "
                          "the others time one component")
     ap.add_argument("--batch", type=int, default=MODEL_CFG["batch"], help="decode batch of --workload model")
@@ -1007,7 +1012,7 @@ def main() -> None:
     ap.add_argument("--cluster", type=int, default=0, help="attn: CTAs per (sequence, KV head); 0 = library default")
     ap.add_argument("--pool-pages", type=int, default=ATTN_CFG["pool_pages"], help="attn: pages in the KV pool")
     ap.add_argument("--rows", type=int, default=16384, help="rows for --workload rowops")
-    ap.add_argument("--sizes", default="", help="sefevik: comma-separated model sizes of bench_hybrid.SIZES; default all")
+    ap.add_argument("--sizes", default="", help="sefevik, derelorn: comma-separated model sizes; default all")
     ap.add_argument("--m", type=int, default=4096, help="M for --workload gemm")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
@@ -1015,7 +1020,7 @@ def main() -> None:
         run_reference(args)
     else:
         {"model": run_model, "attn": run_attn, "rowops": run_rowops, "gemm": run_gemm, "prefill": run_prefill, "offline": run_offline,
-         "tp_layer": run_tp_layer, "tp_linear": run_tp_linear, "sefevik": run_sefevik}[args.workload](args)
+         "tp_layer": run_tp_layer, "tp_linear": run_tp_linear, "sefevik": run_sefevik, "derelorn": run_derelorn}[args.workload](args)
 
 
 if __name__ == "__main__":
