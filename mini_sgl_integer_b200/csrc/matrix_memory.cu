@@ -960,18 +960,19 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     }
 }
 
-// (I + M)^-1 of every chunk and head, as two bf16 panels, and the unit factors of k and q into the gates.
-// A CTA of 4 warps per (chunk, q / k head): k . k on the tensor cores, then a pair of warps per head, a column per thread.
-__global__ void __launch_bounds__(128)
+// (I + M)^-1 of every chunk and head, as two bf16 panels (the 16 x 16 blocks above the diagonal are left undefined), and the
+// unit factors of k and q into the gates.  A CTA of 4 warps per (chunk, q / k head); k . k on the tensor cores once, then head
+// by head: M, the inverses D_i of its four diagonal blocks by substitution, and the blocks below them column by column from
+// T_ij = -D_i sum_(j <= k < i) M_ik T_kj.  The products are transposed as in the chunk kernel, so a block goes from
+// accumulator to left operand in registers; operands are two bf16 numbers each.
+__global__ void __launch_bounds__(128, 4)
 delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* __restrict__ inverse) {
-  extern __shared__ __align__(16) unsigned char smem[];
+  extern __shared__ __align__(128) unsigned char smem[];
   constexpr int C = kChunk;
   const int lk = ((p.dim + 15) & ~15) + 8, k16 = (p.dim + 15) >> 4;
-  float* gm = reinterpret_cast<float*>(smem);            // [C][C] k_t . k_s
-  float* mm = gm + C * C;                                // [2][C][C] M of two heads
-  float* lsum = mm + 2 * C * C;                          // [2][C]
-  float* rk = lsum + 2 * C;                              // [C]
-  float* rq = rk + C;                                    // [C]
+  unsigned char *mp = smem, *tp = smem + 2 * kPanel;     // M and the inverse: a high and a low panel each
+  float* dg = reinterpret_cast<float*>(tp + 2 * kPanel); // [4][16][16] diagonal blocks of M
+  float *ls = dg + 4 * 256, *bs = ls + C, *rk = bs + C, *rq = rk + C;                 // [C] each
   bf16* ks = reinterpret_cast<bf16*>(rq + C);            // [C][lk]
   pdl_launch_dependents();
   pdl_wait();
@@ -980,7 +981,7 @@ delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* 
   const int64_t t0 = p.seq_start[seq];
   const int count = p.seq_start[seq + 1] - (int)t0;
   if (ch * C >= count) return;
-  const int n = min(C, count - ch * C), cq = p.dim / 8;
+  const int n = min(C, count - ch * C), cq = p.dim / 8, per = p.heads / p.qk_heads;
   const int64_t tok = t0 + (int64_t)ch * C;
   const bf16* q_src = rows + tok * p.row_pitch + p.q_off + (int64_t)qh * p.dim;
   const bf16* k_src = rows + tok * p.row_pitch + p.k_off + (int64_t)qh * p.dim;
@@ -993,93 +994,163 @@ delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* 
     for (int c = p.dim; c < lk; ++c) ks[r * lk + c] = __float2bfloat16_rn(0.0f);
   {                                                      // two threads per token
     const int t = tid >> 1;
-    const uint4* src = reinterpret_cast<const uint4*>(q_src + (int64_t)(t < n ? t : 0) * p.row_pitch + (tid & 1) * (p.dim / 2));
-    float ss = 0.0f;
-#pragma unroll 4
-    for (int c = 0; c < p.dim / 16; ++c) {
-      const uint4 v = __ldg(src + c);
+    const int64_t off = (int64_t)(t < n ? t : 0) * p.row_pitch + (tid & 1) * (p.dim / 2);
+    const uint4 *qp = reinterpret_cast<const uint4*>(q_src + off), *kp = reinterpret_cast<const uint4*>(k_src + off);
+    auto squares = [](const uint4& v) {
       const unsigned w[4] = {v.x, v.y, v.z, v.w};
+      float ss = 0.0f;
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float2 x = bf16x2_to_f32(w[k]);
         ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
       }
+      return ss;
+    };
+    float sq = 0.0f, sk = 0.0f;
+#pragma unroll 4
+    for (int c = 0; c < p.dim / 16; ++c) {
+      sq += squares(__ldg(qp + c));
+      sk += squares(__ldg(kp + c));
     }
-    ss += __shfl_xor_sync(FULL_MASK, ss, 1);
-    if ((tid & 1) == 0) rq[t] = p.q_scale / sqrtf(ss + kUnitEps);
+    sq += __shfl_xor_sync(FULL_MASK, sq, 1);
+    sk += __shfl_xor_sync(FULL_MASK, sk, 1);
+    if ((tid & 1) == 0) {
+      rq[t] = p.q_scale / sqrtf(sq + kUnitEps);
+      rk[t] = 1.0f / sqrtf(sk + kUnitEps);
+    }
   }
   cp_async_wait<0>();
   __syncthreads();
-  for (int kb = 0; kb <= warp; ++kb) {
-    float s[2][4] = {};
+  float gm[4][2][4];                                     // this warp's 16 rows of k . k
+#pragma unroll
+  for (int kb = 0; kb < 4; ++kb) {
+    if (kb > warp) break;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) gm[kb][i >> 2][i & 3] = 0.0f;
     for (int kk = 0; kk < k16; ++kk) {
       unsigned a[4], b[4];
       mm_ldsm(a, smem_u32(ks + (warp * 16 + (lane & 15)) * lk + (lane >> 4) * 8 + kk * 16));
       mm_ldsm(b, smem_u32(ks + (kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * lk + ((lane >> 3) & 1) * 8 + kk * 16));
-      mm_mma(s[0], a, b[0], b[1]);
-      mm_mma(s[1], a, b[2], b[3]);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int c = kb * 16 + 8 * i + q2;
-      *reinterpret_cast<float2*>(gm + (warp * 16 + g) * C + c) = make_float2(s[i][0], s[i][1]);
-      *reinterpret_cast<float2*>(gm + (warp * 16 + g + 8) * C + c) = make_float2(s[i][2], s[i][3]);
+      mm_mma(gm[kb][0], a, b[0], b[1]);
+      mm_mma(gm[kb][1], a, b[2], b[3]);
     }
   }
-  __syncthreads();
-  if (tid < C) rk[tid] = 1.0f / sqrtf(gm[tid * C + tid] + kUnitEps);
-  const int per = p.heads / p.qk_heads, wp = warp >> 1, j = tid & 63;
-  float *m = mm + wp * C * C, *l = lsum + wp * C;
-  for (int e0 = 0; e0 < per; e0 += 2) {
-    const int h = qh * per + e0 + wp;
-    const bool live = e0 + wp < per;
-    __syncthreads();                                     // the factors are there; the last heads' M is no longer read
-    float beta = 0.0f;
-    if (live) {
-      const int64_t gi = (tok + (j < n ? j : 0)) * p.heads + h;
-      const float4 gate = j < n ? p.gates[gi] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-      beta = gate.y;
-      if (j < n) {
-        p.gates[gi].z = rk[j];
-        p.gates[gi].w = rq[j];
-      }
-      if ((warp & 1) == 0) {
-        float a = gate.x, b = lane + 32 < n ? p.gates[(tok + lane + 32) * p.heads + h].x : 0.0f;
-        sum64(a, b, lane);
-        l[lane] = a * 1.4426950408889634f;
-        l[lane + 32] = b * 1.4426950408889634f;
+  const unsigned m_base = smem_u32(mp), t_base = smem_u32(tp);
+  const unsigned n_row = ((lane & 7) + ((lane >> 4) << 3)) * 128, n_x = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
+  auto at_n = [&](unsigned base, int row16, int col16) { return base + row16 * 2048 + n_row + (n_x ^ (col16 << 5)); };
+  // d [16, 16] += (ah + al) (b_high + b_low) for a right operand stored [n][k] in block (row16, col16) of a pair of panels
+  auto times = [&](float (&d)[2][4], const unsigned (&ah)[4], const unsigned (&al)[4], unsigned base, int row16, int col16) {
+    unsigned bh[4], bl[4];
+    mm_ldsm(bh, at_n(base, row16, col16));
+    mm_ldsm(bl, at_n(base + kPanel, row16, col16));
+    mm_mma(d[0], ah, bh[0], bh[1]);
+    mm_mma(d[1], ah, bh[2], bh[3]);
+    mm_mma(d[0], al, bh[0], bh[1]);
+    mm_mma(d[1], al, bh[2], bh[3]);
+    mm_mma(d[0], ah, bl[0], bl[1]);
+    mm_mma(d[1], ah, bl[2], bl[3]);
+  };
+  for (int e = 0; e < per; ++e) {
+    const int h = qh * per + e;
+    if (warp == 0) {
+      const float4 z = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      float4* gp = p.gates + (tok + lane) * p.heads + h;
+      const float4 ga = lane < n ? gp[0] : z, gb = lane + 32 < n ? gp[(int64_t)32 * p.heads] : z;
+      float a = ga.x * 1.4426950408889634f, b = gb.x * 1.4426950408889634f;
+      sum64(a, b, lane);
+      ls[lane] = a; ls[lane + 32] = b;
+      bs[lane] = ga.y; bs[lane + 32] = gb.y;
+      if (lane < n) { gp[0].z = rk[lane]; gp[0].w = rq[lane]; }
+      if (lane + 32 < n) { gp[(int64_t)32 * p.heads].z = rk[lane + 32]; gp[(int64_t)32 * p.heads].w = rq[lane + 32]; }
+    }
+    __syncthreads();
+    const int ra = warp * 16 + g;
+    const float la = ls[ra], lb = ls[ra + 8], fa = bs[ra] * rk[ra], fb = bs[ra + 8] * rk[ra + 8];
+#pragma unroll
+    for (int kb = 0; kb < 4; ++kb) {
+      if (kb > warp) break;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int c = kb * 16 + 8 * i + q2;
+        const float2 l = *reinterpret_cast<const float2*>(ls + c), r = *reinterpret_cast<const float2*>(rk + c);
+        const float (&s)[4] = gm[kb][i];
+        float s0 = s[0] * fa * r.x * exp2_fast(la - l.x), s1 = s[1] * fa * r.y * exp2_fast(la - l.y);
+        float s2 = s[2] * fb * r.x * exp2_fast(lb - l.x), s3 = s[3] * fb * r.y * exp2_fast(lb - l.y);
+        if (kb < warp) {
+          unsigned hi, lo;
+          unsigned char* at = mp + ra * 128 + (((kb * 2 + i) ^ g) << 4) + 2 * q2;       // (row ra + 8 has the same last bits)
+          split2(s0, s1, &hi, &lo);
+          *reinterpret_cast<unsigned*>(at) = hi;
+          *reinterpret_cast<unsigned*>(at + kPanel) = lo;
+          split2(s2, s3, &hi, &lo);
+          *reinterpret_cast<unsigned*>(at + 8 * 128) = hi;
+          *reinterpret_cast<unsigned*>(at + 8 * 128 + kPanel) = lo;
+        } else {
+          float* at = dg + kb * 256 + g * 16 + 8 * i + q2;                              // entries above the diagonal are not read
+          *reinterpret_cast<float2*>(at) = make_float2(s0, s1);
+          *reinterpret_cast<float2*>(at + 128) = make_float2(s2, s3);
+        }
       }
     }
     __syncthreads();
-    if (live) {                                          // row j of M
-      const float lj = l[j], f = beta * rk[j];
-      for (int s = 0; s < C; ++s) {
-        const int c = (s + j) & 63;                      // rows start at different banks
-        m[j * C + c] = c < j ? f * rk[c] * gm[j * C + c] * exp2_fast(lj - l[c]) : 0.0f;
-      }
-    }
-    __syncthreads();
-    if (live) {                                          // column j of the inverse, row by row
-      unsigned char* dst = reinterpret_cast<unsigned char*>(inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C));
-      float x[C];
+    if (tid < C) {                                       // column c of a diagonal block's inverse
+      const int b = tid >> 4, c = tid & 15;
+      const float* m = dg + b * 256;
+      float x[16];
 #pragma unroll
-      for (int t = 0; t < C; ++t) {
-        float a0 = t == j ? 1.0f : 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
+      for (int t = 0; t < 16; ++t) {
+        float a0 = t == c ? 1.0f : 0.0f, a1 = 0.0f;
 #pragma unroll
-        for (int s = 0; s < t; s += 4) {
-          const float4 v = *reinterpret_cast<const float4*>(m + t * C + s);
+        for (int s = 0; s < t; s += 2) {
+          const float2 v = *reinterpret_cast<const float2*>(m + t * 16 + s);
           a0 = fmaf(-v.x, x[s], a0);
           if (s + 1 < t) a1 = fmaf(-v.y, x[s + 1], a1);
-          if (s + 2 < t) a2 = fmaf(-v.z, x[s + 2], a2);
-          if (s + 3 < t) a3 = fmaf(-v.w, x[s + 3], a3);
         }
-        x[t] = (a0 + a1) + (a2 + a3);
+        x[t] = a0 + a1;
         const bf16 hi = __float2bfloat16_rn(x[t]);
-        bf16* at = reinterpret_cast<bf16*>(dst + panel_at(t, j));
+        bf16* at = reinterpret_cast<bf16*>(tp + panel_at(b * 16 + t, b * 16 + c));
         at[0] = hi;
         at[C * C] = __float2bfloat16_rn(x[t] - __bfloat162float(hi));
       }
     }
+    __syncthreads();
+    if (warp < 3) {                                      // block column `warp`
+      unsigned th[3][4], tl[3][4];                       // T_kj transposed, as left operands
+      mm_ldsm_t(th[0], at_n(t_base, warp, warp));
+      mm_ldsm_t(tl[0], at_n(t_base + kPanel, warp, warp));
+#pragma unroll
+      for (int d = 1; d < 4; ++d) {
+        const int i = warp + d;
+        if (i >= 4) break;
+        float x[2][4] = {}, y[2][4] = {};
+#pragma unroll
+        for (int k = 0; k < d; ++k) times(x, th[k], tl[k], m_base, i, warp + k);
+        unsigned xh[4], xl[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) split2(-x[k >> 1][2 * (k & 1)], -x[k >> 1][2 * (k & 1) + 1], &xh[k], &xl[k]);
+        times(y, xh, xl, t_base, i, i);
+        unsigned yh[4], yl[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          split2(y[k >> 1][2 * (k & 1)], y[k >> 1][2 * (k & 1) + 1], &yh[k], &yl[k]);
+          // rows of T: 8 (k >> 1) + q2 and the next; column: g + 8 (k & 1)
+          const int row = i * 16 + 8 * (k >> 1) + q2, col = warp * 16 + g + 8 * (k & 1);
+          *reinterpret_cast<unsigned short*>(tp + panel_at(row, col)) = (unsigned short)yh[k];
+          *reinterpret_cast<unsigned short*>(tp + panel_at(row + 1, col)) = (unsigned short)(yh[k] >> 16);
+          *reinterpret_cast<unsigned short*>(tp + kPanel + panel_at(row, col)) = (unsigned short)yl[k];
+          *reinterpret_cast<unsigned short*>(tp + kPanel + panel_at(row + 1, col)) = (unsigned short)(yl[k] >> 16);
+        }
+        if (d < 3) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) { th[d][k] = yh[k]; tl[d][k] = yl[k]; }
+        }
+      }
+    }
+    __syncthreads();
+    uint4* dst = reinterpret_cast<uint4*>(inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C));
+#pragma unroll
+    for (int i = 0; i < 2 * kPanel / 16 / 128; ++i) dst[tid + 128 * i] = *reinterpret_cast<const uint4*>(tp + (tid + 128 * i) * 16);
+    __syncthreads();                                     // the panels may be replaced
   }
 }
 
@@ -1368,7 +1439,7 @@ static int launch_chunks(const MemoryParams& p, const bf16* rows, bf16* inverse,
                  B200_E_CUDA, "memory_scan: cuTensorMapEncodeTiled failed");
   }
   if (KIND == B200F_MEMORY_DELTA) {
-    const size_t bytes = (size_t)3 * kChunk * kChunk * 4 + 4 * kChunk * 4 + (size_t)kChunk * (((p.dim + 15) & ~15) + 8) * 2;
+    const size_t bytes = (size_t)4 * kPanel + 4 * 256 * 4 + 4 * kChunk * 4 + (size_t)kChunk * (((p.dim + 15) & ~15) + 8) * 2;
     cudaError_t e = cudaFuncSetAttribute(delta_inverse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
     B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     launch_pdl(delta_inverse_kernel, dim3((unsigned)((max_q + kChunk - 1) / kChunk), (unsigned)p.qk_heads, (unsigned)batch), dim3(128), bytes, st, p, rows, inverse);
