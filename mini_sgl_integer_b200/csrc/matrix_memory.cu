@@ -507,7 +507,8 @@ running_max_kernel(const MemoryPrepare p) {
 // A CTA per (sequence, head, 64 columns); each of 4 warps owns 16 columns and holds S^T [16, dim] in accumulators over all
 // chunks.  With everything transposed, an accumulator tile has the layout of the left operand of the next product, so S, the
 // right-hand side and U never leave the registers; shared memory holds q, k, v, the decayed scores and the inverse, each
-// read as the right operand.  EXP: in the CTA of the first columns a fifth warp's first column is n, written by ones.
+// read as the right operand.  EXP: the CTA of the first columns also runs the normaliser, n . q = e^L (n_0 . q) + the row sums
+// of the decayed scores, on the fp32 units.
 // ---------------------------------------------------------------------------------------------------
 constexpr int kChunk = 64, kChunkWarps = 4, kChunkCols = 16 * kChunkWarps;
 constexpr int kPanel = kChunk * 128;     // bytes of 64 rows of 64 bf16 values, as TMA writes them with the 128-byte swizzle
@@ -551,8 +552,9 @@ __device__ __forceinline__ void async_fence() { asm volatile("fence.proxy.async.
 __device__ __forceinline__ int64_t chunk_index(int64_t first_token, int seq, int chunk) { return first_token / kChunk + seq + chunk; }
 
 __host__ __device__ constexpr int chunk_panels(int dr) { return dr <= 4 ? 1 : dr / 4; }
-__host__ __device__ constexpr size_t chunk_smem(int dr, bool delta) {
-  return (size_t)(2 * chunk_panels(dr) + (delta ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 2 * kChunk * 16 + 8 + 1024;
+__host__ __device__ constexpr size_t chunk_smem(int dr, int kind) {
+  return (size_t)(2 * chunk_panels(dr) + (kind == B200F_MEMORY_DELTA ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 2 * kChunk * 16 +
+         (kind == B200F_MEMORY_EXP ? (9 * 16 * dr + 4 * kChunk) * 4 : 0) + 8 + 1024;
 }
 // Byte offset of (row, col) in a panel.
 __host__ __device__ __forceinline__ int panel_at(int row, int col) { return row * 128 + ((((col >> 3) ^ row) & 7) << 4) + (col & 7) * 2; }
@@ -568,11 +570,11 @@ __device__ __forceinline__ void sum64(float& a, float& b, int lane) {
 }
 
 template <int KIND, int DR, bool FULL>      // FULL: dim is exactly 16 DR
-__global__ void __launch_bounds__(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0), DR > 8 ? 1 : (DR == 8 && KIND == B200F_MEMORY_EXP ? 2 : 3))
+__global__ void __launch_bounds__(kChunkWarps * 32, DR > 8 ? 1 : 2)
 memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams p, const bf16* __restrict__ inverse) {
   extern __shared__ __align__(16) unsigned char smem[];
   constexpr bool DELTA = KIND == B200F_MEMORY_DELTA, EXP = KIND == B200F_MEMORY_EXP;
-  constexpr int C = kChunk, NW = kChunkWarps, THREADS = NW * 32 + (EXP ? 32 : 0), DP = chunk_panels(DR);
+  constexpr int C = kChunk, THREADS = kChunkWarps * 32, DP = chunk_panels(DR);
   // panels: q [DP], k [DP], v, then the decayed scores' low and high parts (DELTA: the high part takes the place of v, which is
   // used up by then) and, DELTA, the inverse's high and low parts
   const unsigned q_base = (smem_u32(smem) + 1023) & ~1023u, k_base = q_base + DP * kPanel, v_base = k_base + DP * kPanel;
@@ -586,7 +588,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
   const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, col0 = slice * kChunkCols;
   const int vp = p.vdim, k16 = p.dim >> 4, qh = h / (p.heads / p.qk_heads);
   float4* gs = reinterpret_cast<float4*>(es + C);        // [2][C]
-  const unsigned bar = smem_u32(gs + 2 * C);
+  float *ns = reinterpret_cast<float*>(gs + 2 * C), *nsum = ns + (EXP ? 16 * DR : 0), *np = nsum + (EXP ? 4 * C : 0);   // EXP: n, row sums of the scores by column block, parts of n's update
+  const unsigned bar = smem_u32(np + (EXP ? 8 * 16 * DR : 0));
   if (tid == 0) {
     mbar_init(bar, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -597,8 +600,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
   const int count = p.seq_start[seq + 1] - (int)t0;
   if (count <= 0) return;
   const bool has_state = p.positions[t0] > 0;
-  const bool is_n = EXP && warp == NW;                   // this warp's first column is the normaliser
-  const bool works = is_n ? slice == 0 : col0 + warp * 16 < vp;
+  const bool with_n = EXP && slice == 0, works = col0 + warp * 16 < vp;
   const int64_t slot_head = (int64_t)p.slots[seq] * p.heads + h;
   const int64_t q_col = p.q_off + (int64_t)qh * p.dim, k_col = p.k_off + (int64_t)qh * p.dim, v_col = p.v_off + (int64_t)h * vp + col0;
 
@@ -616,13 +618,14 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
       float v = 0.0f;
       if (has_state && works && (FULL || d < p.dim)) {
-        if (is_n) v = k < 2 && g == 0 ? nst[d] : 0.0f;
-        else if (col0 + c < vp) v = st[(int64_t)d * vp + c];
+        if (col0 + c < vp) v = st[(int64_t)d * vp + c];
       }
       S[i][k] = v;
     }
 
   // ldmatrix addresses: rows of 128 bytes, 16-byte pieces exchanged by the row's last three bits
+  if (with_n)
+    for (int d = tid; d < 16 * DR; d += THREADS) ns[d] = has_state && d < p.dim ? nst[d] : 0.0f;
   const unsigned n_row = ((lane & 7) + ((lane >> 4) << 3)) * 128, n_x = (((lane >> 3) & 1) ^ (lane & 7)) << 4;     // right operand from [n][k], left from [k][m]
   const unsigned m_row = (lane & 15) * 128, m_x = ((lane >> 4) ^ (lane & 7)) << 4;                                 // left operand from [m][k], right from [k][n]
   unsigned n_at[4], m_at[4];
@@ -663,14 +666,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     }
   };
   // V^T of 16 tokens as a left operand; in the accumulator layout: pairs of tokens
-  auto values = [&](int kb, unsigned (&a)[4]) {
-    if (is_n) {
-      a[0] = a[2] = g == 0 ? 0x3f803f80u : 0u;           // ones
-      a[1] = a[3] = 0u;
-    } else {
-      mm_ldsm_t(a, v_at + kb * 2048);
-    }
-  };
+  auto values = [&](int kb, unsigned (&a)[4]) { mm_ldsm_t(a, v_at + kb * 2048); };
 
   const int chunks = (count + C - 1) / C;
   auto load_gates = [&](int ch) {                         // by warp 0, a chunk ahead; entries behind the portion are not used
@@ -781,6 +777,38 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       __syncthreads();                                    // the values' place is taken by the scores
     }
 
+    float q_n = 0.0f;                                     // two threads per token: q . n in front of the chunk
+    if (with_n) {
+      const int t = tid >> 1, half = tid & 1;
+      for (int c = half; c < k16 * 2; c += 2) {           // pieces of 8 values
+        const uint4 x = *reinterpret_cast<const uint4*>(panels + (c >> 3) * kPanel + t * 128 + (((c ^ t) & 7) << 4));
+        const float4 n0 = *reinterpret_cast<const float4*>(ns + 8 * c), n1 = *reinterpret_cast<const float4*>(ns + 8 * c + 4);
+        const float2 x0 = bf16x2_to_f32(x.x), x1 = bf16x2_to_f32(x.y), x2 = bf16x2_to_f32(x.z), x3 = bf16x2_to_f32(x.w);
+        q_n = fmaf(x0.x, n0.x, fmaf(x0.y, n0.y, fmaf(x1.x, n0.z, fmaf(x1.y, n0.w, q_n))));
+        q_n = fmaf(x2.x, n1.x, fmaf(x2.y, n1.y, fmaf(x3.x, n1.z, fmaf(x3.y, n1.w, q_n))));
+      }
+      q_n += __shfl_xor_sync(FULL_MASK, q_n, 1);
+      for (int i = tid; i < 16 * k16; i += THREADS) {     // sums of 8 decayed keys, 8 entries of each
+        const int c = i >> 3, tg = i & 7;
+        float acc[8] = {};
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          const uint4 x = *reinterpret_cast<const uint4*>(panels + (DP + (c >> 3)) * kPanel + (8 * tg + u) * 128 + (((c ^ u) & 7) << 4));
+          const unsigned w[4] = {x.x, x.y, x.z, x.w};
+          const float e = es[8 * tg + u];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 f = bf16x2_to_f32(w[k]);
+            acc[2 * k] = fmaf(e, f.x, acc[2 * k]);
+            acc[2 * k + 1] = fmaf(e, f.y, acc[2 * k + 1]);
+          }
+        }
+        float4* dst = reinterpret_cast<float4*>(np + tg * 16 * DR + 8 * c);
+        dst[0] = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        dst[1] = make_float4(acc[4], acc[5], acc[6], acc[7]);
+      }
+    }
+
     // decayed scores: the ten 16 x 16 blocks on and below the diagonal
     constexpr int WARPS = THREADS / 32, MINE = (10 + WARPS - 1) / WARPS;
     float sc[MINE][2][4];
@@ -812,6 +840,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       float (&s)[2][4] = sc[m];
       const int ra = rb * 16 + g;
       const float la = ls[ra], lb = ls[ra + 8];
+      float sum_a = 0.0f, sum_b = 0.0f;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int c = kb * 16 + 8 * i + q2;
@@ -823,6 +852,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         s1 = c < ra ? s1 : 0.0f;
         s2 = c <= ra + 8 ? s2 : 0.0f;
         s3 = c < ra + 8 ? s3 : 0.0f;
+        sum_a += s0 + s1;
+        sum_b += s2 + s3;
         unsigned hi, lo;
         split2(s0, s1, &hi, &lo);
         unsigned char* at = panels + ra * 128 + (((kb * 2 + i) ^ g) << 4) + 2 * q2;     // (row ra + 8 has the same last bits)
@@ -832,8 +863,33 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         *reinterpret_cast<unsigned*>(at + (ph_base - q_base) + 8 * 128) = hi;
         *reinterpret_cast<unsigned*>(at + (pl_base - q_base) + 8 * 128) = lo;
       }
+      if (with_n) {
+#pragma unroll
+        for (int o = 1; o < 4; o <<= 1) {
+          sum_a += __shfl_xor_sync(FULL_MASK, sum_a, o);
+          sum_b += __shfl_xor_sync(FULL_MASK, sum_b, o);
+        }
+        if (q2 == 0) {
+          nsum[kb * C + ra] = sum_a;
+          nsum[kb * C + ra + 8] = sum_b;
+        }
+      }
     }
     __syncthreads();
+    if (with_n) {
+      const int t = tid >> 1;
+      if ((tid & 1) == 0 && t < n) {
+        float dot = q_n * el[t];
+        for (int kb = 0; kb <= t >> 4; ++kb) dot += nsum[kb * C + t];
+        p.den[(tok + t) * p.heads + h] = fmaxf(fabsf(dot * rs[t]), zs[t]) + kUnitEps;
+      }
+      for (int d = tid; d < 16 * k16; d += THREADS) {
+        float v = ns[d] * el[C - 1];
+#pragma unroll
+        for (int tg = 0; tg < 8; ++tg) v += np[tg * 16 * DR + d];
+        ns[d] = v;
+      }
+    }
 
     if (works) {
       float o[8][4] = {};
@@ -916,17 +972,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
           }
         }
       }
-      if (is_n) {
-        if (g == 0) {
-#pragma unroll
-          for (int i = 0; i < 8; ++i)
-#pragma unroll
-            for (int k = 0; k < 2; ++k) {
-              const int t = i * 8 + q2 + k;
-              if (t < n) p.den[(tok + t) * p.heads + h] = fmaxf(fabsf(o[i][k] * rs[t]), zs[t]) + kUnitEps;
-            }
-        }
-      } else {
+      {
         const int64_t pitch = (int64_t)p.heads * p.vdim;
         float* out = p.out + (tok + q2) * pitch + (int64_t)h * p.vdim + col0 + c_lo;
         const bool lo = col0 + c_lo < vp, hi = col0 + c_hi < vp;
@@ -945,6 +991,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     async_fence();
     __syncthreads();                                       // everything in shared memory may be replaced
   }
+  if (with_n)
+    for (int d = tid; d < p.dim; d += THREADS) nst[d] = ns[d];
   if (!works) return;
 #pragma unroll
   for (int i = 0; i < 2 * DR; ++i)
@@ -952,11 +1000,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     for (int k = 0; k < 4; ++k) {
       const int d = i * 8 + q2 + (k & 1), c = k < 2 ? c_lo : c_hi;
       if (!FULL && d >= p.dim) continue;
-      if (is_n) {
-        if (k < 2 && g == 0) nst[d] = S[i][k];
-      } else if (col0 + c < vp) {
-        st[(int64_t)d * vp + c] = S[i][k];
-      }
+      if (col0 + c < vp) st[(int64_t)d * vp + c] = S[i][k];
     }
 }
 
@@ -1418,12 +1462,12 @@ static int launch_scan_shape(MemoryParams p, const T* rows, int batch, cudaStrea
 }
 template <int KIND, int DR, bool FULL>
 static int launch_chunk_shape(const CUtensorMap& map, const MemoryParams& p, const bf16* inverse, int batch, cudaStream_t st) {
-  constexpr size_t bytes = chunk_smem(DR, KIND == B200F_MEMORY_DELTA);
+  constexpr size_t bytes = chunk_smem(DR, KIND);
   static_assert(bytes <= 227 * 1024, "shared memory budget");
   cudaError_t e = cudaFuncSetAttribute(memory_chunk_kernel<KIND, DR, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
   B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
   const dim3 grid((unsigned)((p.vdim + kChunkCols - 1) / kChunkCols), (unsigned)p.heads, (unsigned)batch);
-  launch_pdl(memory_chunk_kernel<KIND, DR, FULL>, grid, dim3(kChunkWarps * 32 + (KIND == B200F_MEMORY_EXP ? 32 : 0)), bytes, st, map, p, inverse);
+  launch_pdl(memory_chunk_kernel<KIND, DR, FULL>, grid, dim3(kChunkWarps * 32), bytes, st, map, p, inverse);
   return check_launch("memory_scan (chunks)");
 }
 template <int KIND>
