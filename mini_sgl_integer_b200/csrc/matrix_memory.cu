@@ -780,16 +780,25 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     float q_n = 0.0f;                                     // two threads per token: q . n in front of the chunk
     if (with_n) {
       const int t = tid >> 1, half = tid & 1;
-      for (int c = half; c < k16 * 2; c += 2) {           // pieces of 8 values
+      float acc[4] = {};
+#pragma unroll
+      for (int i = 0; i < DR; ++i) {                      // pieces of 8 values
+        if (!FULL && i >= k16) break;
+        const int c = 2 * i + half;
         const uint4 x = *reinterpret_cast<const uint4*>(panels + (c >> 3) * kPanel + t * 128 + (((c ^ t) & 7) << 4));
         const float4 n0 = *reinterpret_cast<const float4*>(ns + 8 * c), n1 = *reinterpret_cast<const float4*>(ns + 8 * c + 4);
         const float2 x0 = bf16x2_to_f32(x.x), x1 = bf16x2_to_f32(x.y), x2 = bf16x2_to_f32(x.z), x3 = bf16x2_to_f32(x.w);
-        q_n = fmaf(x0.x, n0.x, fmaf(x0.y, n0.y, fmaf(x1.x, n0.z, fmaf(x1.y, n0.w, q_n))));
-        q_n = fmaf(x2.x, n1.x, fmaf(x2.y, n1.y, fmaf(x3.x, n1.z, fmaf(x3.y, n1.w, q_n))));
+        acc[0] = fmaf(x0.x, n0.x, fmaf(x0.y, n0.y, acc[0]));
+        acc[1] = fmaf(x1.x, n0.z, fmaf(x1.y, n0.w, acc[1]));
+        acc[2] = fmaf(x2.x, n1.x, fmaf(x2.y, n1.y, acc[2]));
+        acc[3] = fmaf(x3.x, n1.z, fmaf(x3.y, n1.w, acc[3]));
       }
+      q_n = (acc[0] + acc[1]) + (acc[2] + acc[3]);
       q_n += __shfl_xor_sync(FULL_MASK, q_n, 1);
-      for (int i = tid; i < 16 * k16; i += THREADS) {     // sums of 8 decayed keys, 8 entries of each
-        const int c = i >> 3, tg = i & 7;
+#pragma unroll
+      for (int i0 = 0; i0 < 16 * DR; i0 += THREADS) {     // sums of 8 decayed keys, 8 entries of each
+        const int i = i0 + tid, c = i >> 3, tg = i & 7;
+        if (i >= 16 * k16) break;
         float acc[8] = {};
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
@@ -880,7 +889,9 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       const int t = tid >> 1;
       if ((tid & 1) == 0 && t < n) {
         float dot = q_n * el[t];
-        for (int kb = 0; kb <= t >> 4; ++kb) dot += nsum[kb * C + t];
+#pragma unroll
+        for (int kb = 0; kb < 4; ++kb)
+          if (kb <= t >> 4) dot += nsum[kb * C + t];
         p.den[(tok + t) * p.heads + h] = fmaxf(fabsf(dot * rs[t]), zs[t]) + kUnitEps;
       }
       for (int d = tid; d < 16 * k16; d += THREADS) {
