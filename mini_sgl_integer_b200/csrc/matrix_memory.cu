@@ -553,8 +553,8 @@ __device__ __forceinline__ int64_t chunk_index(int64_t first_token, int seq, int
 
 __host__ __device__ constexpr int chunk_panels(int dr) { return dr <= 4 ? 1 : dr / 4; }
 __host__ __device__ constexpr size_t chunk_smem(int dr, int kind) {
-  return (size_t)(2 * chunk_panels(dr) + (kind == B200F_MEMORY_DELTA ? 4 : 3)) * kPanel + 6 * kChunk * 4 + 2 * kChunk * 16 +
-         (kind == B200F_MEMORY_EXP ? (9 * 16 * dr + 4 * kChunk) * 4 : 0) + 8 + 1024;
+  return (size_t)(2 * (2 * chunk_panels(dr) + 1) + (kind == B200F_MEMORY_DELTA ? 3 : 2)) * kPanel + 12 * kChunk * 4 + 2 * kChunk * 16 +
+         (kind == B200F_MEMORY_EXP ? (9 * 16 * dr + 4 * kChunk) * 4 : 0) + 24 + 1024;
 }
 // Byte offset of (row, col) in a panel.
 __host__ __device__ __forceinline__ int panel_at(int row, int col) { return row * 128 + ((((col >> 3) ^ row) & 7) << 4) + (col & 7) * 2; }
@@ -575,23 +575,24 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
   extern __shared__ __align__(16) unsigned char smem[];
   constexpr bool DELTA = KIND == B200F_MEMORY_DELTA, EXP = KIND == B200F_MEMORY_EXP;
   constexpr int C = kChunk, THREADS = kChunkWarps * 32, DP = chunk_panels(DR);
-  // panels: q [DP], k [DP], v, then the decayed scores' low and high parts (DELTA: the high part takes the place of v, which is
-  // used up by then) and, DELTA, the inverse's high and low parts
-  const unsigned q_base = (smem_u32(smem) + 1023) & ~1023u, k_base = q_base + DP * kPanel, v_base = k_base + DP * kPanel;
-  const unsigned pl_base = v_base + kPanel, ph_base = DELTA ? v_base : pl_base + kPanel, t_base = pl_base + kPanel;
-  unsigned char* panels = smem + (q_base - smem_u32(smem));
-  float* ls = reinterpret_cast<float*>(panels + (2 * DP + (DELTA ? 4 : 3)) * kPanel);        // [C] L in units of log2
-  float *el = ls + C, *bs = el + C, *zs = bs + C, *rs = zs + C, *es = rs + C; // e^L; write strength; exp(-m) or 1 / |k|; scale of q; e^(L_64 - L) times b or 1 / |k|
+  // panels: twice (q [DP], k [DP], v), for this chunk and the next, then the decayed scores' low and high parts (DELTA: the high
+  // part takes the place of v, which is used up by then) and, DELTA, the inverse's high and low parts
+  constexpr int K_ = DP, V_ = 2 * DP, NB = 2 * DP + 1, PL_ = 2 * NB, PH_ = DELTA ? V_ : PL_ + 1, T_ = PL_ + 1;
+  const unsigned p_base = (smem_u32(smem) + 1023) & ~1023u;
+  unsigned char* panels = smem + (p_base - smem_u32(smem));
+  // per token, for this chunk and the next: L in units of log2; e^L; write strength; exp(-m) or 1 / |k|; scale of q; e^(L_64 - L)
+  // times the strength or 1 / |k|
+  float* token_values = reinterpret_cast<float*>(panels + (PL_ + (DELTA ? 3 : 2)) * kPanel);
 
   pdl_launch_dependents();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
   const int slice = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, col0 = slice * kChunkCols;
   const int vp = p.vdim, k16 = p.dim >> 4, qh = h / (p.heads / p.qk_heads);
-  float4* gs = reinterpret_cast<float4*>(es + C);        // [2][C]
+  float4* gs = reinterpret_cast<float4*>(token_values + 12 * C);        // [2][C]
   float *ns = reinterpret_cast<float*>(gs + 2 * C), *nsum = ns + (EXP ? 16 * DR : 0), *np = nsum + (EXP ? 4 * C : 0);   // EXP: n, row sums of the scores by column block, parts of n's update
   const unsigned bar = smem_u32(np + (EXP ? 8 * 16 * DR : 0));
   if (tid == 0) {
-    mbar_init(bar, 1);
+    for (int i = 0; i < 3; ++i) mbar_init(bar + 8 * i, 1);                // this chunk, the next; the inverse
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   __syncthreads();
@@ -628,17 +629,16 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     for (int d = tid; d < 16 * DR; d += THREADS) ns[d] = has_state && d < p.dim ? nst[d] : 0.0f;
   const unsigned n_row = ((lane & 7) + ((lane >> 4) << 3)) * 128, n_x = (((lane >> 3) & 1) ^ (lane & 7)) << 4;     // right operand from [n][k], left from [k][m]
   const unsigned m_row = (lane & 15) * 128, m_x = ((lane >> 4) ^ (lane & 7)) << 4;                                 // left operand from [m][k], right from [k][n]
-  unsigned n_at[4], m_at[4];
+  unsigned n_at[4], m_at[4], n_fix[4];                   // in the current chunk's panels, and in those there are one of
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    n_at[i] = q_base + n_row + (n_x ^ (i << 5));
-    m_at[i] = q_base + m_row + (m_x ^ (i << 5));
+    n_fix[i] = n_at[i] = p_base + n_row + (n_x ^ (i << 5));
+    m_at[i] = p_base + m_row + (m_x ^ (i << 5));
   }
-  // `panel`: number of a panel from q's first on
+  unsigned v_at = p_base + V_ * kPanel + n_row + (n_x ^ ((warp & 3) << 5));
   auto at_n = [&](int panel, int row16, int k16th) { return n_at[k16th & 3] + (panel + (k16th >> 2)) * kPanel + row16 * 2048; };
   auto at_m = [&](int panel, int row16, int k16th) { return m_at[k16th & 3] + (panel + (k16th >> 2)) * kPanel + row16 * 2048; };
-  constexpr int Q_ = 0, K_ = DP, V_ = 2 * DP, PL_ = V_ + 1, PH_ = DELTA ? V_ : PL_ + 1, T_ = PL_ + 1;
-  const unsigned v_at = q_base + V_ * kPanel + n_row + (n_x ^ ((warp & 3) << 5));
+  auto at_fix = [&](int panel, int row16, int k16th) { return n_fix[k16th & 3] + (panel + (k16th >> 2)) * kPanel + row16 * 2048; };
 
   // acc [16 columns, 64 tokens] = S^T X^T for X = q or k
   auto state_times = [&](int x, float (&acc)[8][4]) {
@@ -677,22 +677,26 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     }
     cp_async_commit();
   };
+  auto load_chunk = [&](int ch) {                         // by one thread
+    const unsigned to = p_base + (ch & 1) * NB * kPanel, b = bar + 8 * (ch & 1);
+    const int tok = (int)(t0 + (int64_t)ch * C);
+    mbar_expect_tx(b, NB * kPanel);
+#pragma unroll
+    for (int d = 0; d < DP; ++d) {
+      tma_load_2d(to + d * kPanel, &map, (int)q_col + 64 * d, tok, b);
+      tma_load_2d(to + (K_ + d) * kPanel, &map, (int)k_col + 64 * d, tok, b);
+    }
+    tma_load_2d(to + V_ * kPanel, &map, (int)v_col, tok, b);
+  };
+  if (tid == 32) load_chunk(0);
   if (warp == 0) load_gates(0);
   for (int ch = 0; ch < chunks; ++ch) {
     const int n = min(C, count - ch * C);
     const int64_t tok = t0 + (int64_t)ch * C;
+    float* ls = token_values + (ch & 1) * 6 * C;
+    float *el = ls + C, *bs = el + C, *zs = bs + C, *rs = zs + C, *es = rs + C;
+    unsigned char* cur = panels + (ch & 1) * NB * kPanel;
     if (warp == 0) {
-      if (lane == 0) {
-        mbar_expect_tx(bar, (2 * DP + 1) * kPanel + (DELTA ? 2 * kPanel : 0));
-#pragma unroll
-        for (int d = 0; d < DP; ++d) {
-          tma_load_2d(q_base + d * kPanel, &map, (int)q_col + 64 * d, (int)tok, bar);
-          tma_load_2d(k_base + d * kPanel, &map, (int)k_col + 64 * d, (int)tok, bar);
-        }
-        tma_load_2d(v_base, &map, (int)v_col, (int)tok, bar);
-        if (DELTA) bulk_copy(t_base, inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C), 2 * kPanel, bar);
-      }
-      __syncwarp();
       load_gates(ch + 1);
       cp_async_wait<1>();
       __syncwarp();
@@ -708,20 +712,31 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       rs[lane] = DELTA ? ga.w : p.q_scale; rs[lane + 32] = DELTA ? gb.w : p.q_scale;
       es[lane] = exp2_fast(last - la) * (DELTA ? ga.z : ga.y); es[lane + 32] = exp2_fast(last - lb) * (DELTA ? gb.z : gb.y);
     }
-    if (__syncthreads_or(!mbar_wait(bar, ch & 1, 7))) {    // expired (the status word says so): once more for the copies, and out
-      mbar_wait(bar, ch & 1, 7);
+    async_fence();
+    // every warp is done with the chunk before: its panels may be replaced
+    const bool late = !mbar_wait(bar + 8 * (ch & 1), (ch >> 1) & 1, 7);
+    if (__syncthreads_or(late)) {                          // expired (the status word says so): once more for the copies, and out
+      mbar_wait(bar + 8 * (ch & 1), (ch >> 1) & 1, 7);
       return;
+    }
+    if (tid == 32) {
+      if (DELTA) {
+        mbar_expect_tx(bar + 16, 2 * kPanel);
+        bulk_copy(p_base + T_ * kPanel, inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C), 2 * kPanel, bar + 16);
+      }
+      if (ch + 1 < chunks) load_chunk(ch + 1);
     }
     if (n < C) {                                          // behind the portion: k and v of other sequences, to be zero here
       for (int i = tid; i < (C - n) * 8 * (DP + 1); i += THREADS) {
         const int r = n + i / (8 * (DP + 1)), c = i % (8 * (DP + 1));
-        *reinterpret_cast<uint4*>(panels + (DP + (c >> 3)) * kPanel + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+        *reinterpret_cast<uint4*>(cur + (K_ + (c >> 3)) * kPanel + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
       }
       __syncthreads();
     }
 
     float u[8][4];                                        // DELTA: U^T
     if (DELTA) {
+      bool there = true;
       if (works) {
         float r[8][4] = {};                               // right-hand side beta (v - e^L K S_0), transposed
         state_times(K_, r);
@@ -740,6 +755,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
             a[2] = b0 * (y.x - f0 * a[2]); a[3] = b1 * (y.y - f1 * a[3]);
           }
         }
+        there = mbar_wait(bar + 16, ch & 1, 7);
 #pragma unroll
         for (int i = 0; i < 8; ++i)
 #pragma unroll
@@ -754,8 +770,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
           unsigned bh[4][4], bl[4][4];
 #pragma unroll
           for (int j = kb; j < 4; ++j) {
-            mm_ldsm(bh[j], at_n(T_, j, kb));
-            mm_ldsm(bl[j], at_n(T_ + 1, j, kb));
+            mm_ldsm(bh[j], at_fix(T_, j, kb));
+            mm_ldsm(bl[j], at_fix(T_ + 1, j, kb));
           }
 #pragma unroll
           for (int j = kb; j < 4; ++j) {
@@ -774,7 +790,11 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
           }
         }
       }
-      __syncthreads();                                    // the values' place is taken by the scores
+      if (__syncthreads_or(!there)) {                     // (the values' place is taken by the scores)
+        mbar_wait(bar + 16, ch & 1, 7);
+        if (ch + 1 < chunks) mbar_wait(bar + 8 * ((ch + 1) & 1), ((ch + 1) >> 1) & 1, 7);
+        return;
+      }
     }
 
     float q_n = 0.0f;                                     // two threads per token: q . n in front of the chunk
@@ -785,7 +805,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       for (int i = 0; i < DR; ++i) {                      // pieces of 8 values
         if (!FULL && i >= k16) break;
         const int c = 2 * i + half;
-        const uint4 x = *reinterpret_cast<const uint4*>(panels + (c >> 3) * kPanel + t * 128 + (((c ^ t) & 7) << 4));
+        const uint4 x = *reinterpret_cast<const uint4*>(cur + (c >> 3) * kPanel + t * 128 + (((c ^ t) & 7) << 4));
         const float4 n0 = *reinterpret_cast<const float4*>(ns + 8 * c), n1 = *reinterpret_cast<const float4*>(ns + 8 * c + 4);
         const float2 x0 = bf16x2_to_f32(x.x), x1 = bf16x2_to_f32(x.y), x2 = bf16x2_to_f32(x.z), x3 = bf16x2_to_f32(x.w);
         acc[0] = fmaf(x0.x, n0.x, fmaf(x0.y, n0.y, acc[0]));
@@ -802,7 +822,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         float acc[8] = {};
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
-          const uint4 x = *reinterpret_cast<const uint4*>(panels + (DP + (c >> 3)) * kPanel + (8 * tg + u) * 128 + (((c ^ u) & 7) << 4));
+          const uint4 x = *reinterpret_cast<const uint4*>(cur + (K_ + (c >> 3)) * kPanel + (8 * tg + u) * 128 + (((c ^ u) & 7) << 4));
           const unsigned w[4] = {x.x, x.y, x.z, x.w};
           const float e = es[8 * tg + u];
 #pragma unroll
@@ -832,7 +852,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
 #pragma unroll
       for (int m = 0; m < MINE; ++m) {
         const int blk = min(warp + m * WARPS, 9), rb = (blk >= 1) + (blk >= 3) + (blk >= 6), kb = blk - rb * (rb + 1) / 2;
-        mm_ldsm(a[m], at_m(Q_, rb, kk));
+        mm_ldsm(a[m], at_m(0, rb, kk));
         mm_ldsm(b[m], at_n(K_, kb, kk));
       }
 #pragma unroll
@@ -865,12 +885,13 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         sum_b += s2 + s3;
         unsigned hi, lo;
         split2(s0, s1, &hi, &lo);
-        unsigned char* at = panels + ra * 128 + (((kb * 2 + i) ^ g) << 4) + 2 * q2;     // (row ra + 8 has the same last bits)
-        *reinterpret_cast<unsigned*>(at + (ph_base - q_base)) = hi;
-        *reinterpret_cast<unsigned*>(at + (pl_base - q_base)) = lo;
+        const int to = ra * 128 + (((kb * 2 + i) ^ g) << 4) + 2 * q2;                  // (row ra + 8 has the same last bits)
+        unsigned char *hp = (DELTA ? cur : panels) + PH_ * kPanel + to, *lp = panels + PL_ * kPanel + to;
+        *reinterpret_cast<unsigned*>(hp) = hi;
+        *reinterpret_cast<unsigned*>(lp) = lo;
         split2(s2, s3, &hi, &lo);
-        *reinterpret_cast<unsigned*>(at + (ph_base - q_base) + 8 * 128) = hi;
-        *reinterpret_cast<unsigned*>(at + (pl_base - q_base) + 8 * 128) = lo;
+        *reinterpret_cast<unsigned*>(hp + 8 * 128) = hi;
+        *reinterpret_cast<unsigned*>(lp + 8 * 128) = lo;
       }
       if (with_n) {
 #pragma unroll
@@ -904,7 +925,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
 
     if (works) {
       float o[8][4] = {};
-      state_times(Q_, o);
+      state_times(0, o);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const float2 e = *reinterpret_cast<const float2*>(el + i * 8 + q2);
@@ -944,8 +965,8 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         unsigned bh[4][4], bl[4][4];
 #pragma unroll
         for (int j = kb; j < 4; ++j) {
-          mm_ldsm(bh[j], at_n(PH_, j, kb));
-          mm_ldsm(bl[j], at_n(PL_, j, kb));
+          mm_ldsm(bh[j], DELTA ? at_n(PH_, j, kb) : at_fix(PH_, j, kb));
+          mm_ldsm(bl[j], at_fix(PL_, j, kb));
         }
 #pragma unroll
         for (int j = kb; j < 4; ++j) {
@@ -999,9 +1020,15 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
         }
       }
     }
-    async_fence();
-    __syncthreads();                                       // everything in shared memory may be replaced
+    const unsigned other = ch & 1 ? 0u - NB * kPanel : NB * kPanel;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      n_at[i] += other;
+      m_at[i] += other;
+    }
+    v_at += other;
   }
+  __syncthreads();
   if (with_n)
     for (int d = tid; d < p.dim; d += THREADS) nst[d] = ns[d];
   if (!works) return;
