@@ -677,18 +677,20 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
     }
     cp_async_commit();
   };
-  auto load_chunk = [&](int ch) {                         // by one thread
+  auto load_chunk = [&](int ch) {                         // by the first lane of every warp: an issue takes long, so they share
     const unsigned to = p_base + (ch & 1) * NB * kPanel, b = bar + 8 * (ch & 1);
     const int tok = (int)(t0 + (int64_t)ch * C);
-    mbar_expect_tx(b, NB * kPanel);
+    if (warp == 1) {
+      mbar_expect_tx(b, NB * kPanel);
+      tma_load_2d(to + V_ * kPanel, &map, (int)v_col, tok, b);
+    }
 #pragma unroll
     for (int d = 0; d < DP; ++d) {
-      tma_load_2d(to + d * kPanel, &map, (int)q_col + 64 * d, tok, b);
-      tma_load_2d(to + (K_ + d) * kPanel, &map, (int)k_col + 64 * d, tok, b);
+      if (warp == ((2 + 2 * d) & 3)) tma_load_2d(to + d * kPanel, &map, (int)q_col + 64 * d, tok, b);
+      if (warp == ((3 + 2 * d) & 3)) tma_load_2d(to + (K_ + d) * kPanel, &map, (int)k_col + 64 * d, tok, b);
     }
-    tma_load_2d(to + V_ * kPanel, &map, (int)v_col, tok, b);
   };
-  if (tid == 32) load_chunk(0);
+  if (lane == 0) load_chunk(0);
   if (warp == 0) load_gates(0);
   for (int ch = 0; ch < chunks; ++ch) {
     const int n = min(C, count - ch * C);
@@ -712,15 +714,15 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       rs[lane] = DELTA ? ga.w : p.q_scale; rs[lane + 32] = DELTA ? gb.w : p.q_scale;
       es[lane] = exp2_fast(last - la) * (DELTA ? ga.z : ga.y); es[lane + 32] = exp2_fast(last - lb) * (DELTA ? gb.z : gb.y);
     }
-    async_fence();
+    if (DELTA) async_fence();                              // (the scores were written over the values)
     // every warp is done with the chunk before: its panels may be replaced
     const bool late = !mbar_wait(bar + 8 * (ch & 1), (ch >> 1) & 1, 7);
     if (__syncthreads_or(late)) {                          // expired (the status word says so): once more for the copies, and out
       mbar_wait(bar + 8 * (ch & 1), (ch >> 1) & 1, 7);
       return;
     }
-    if (tid == 32) {
-      if (DELTA) {
+    if (lane == 0) {
+      if (DELTA && warp == 0) {
         mbar_expect_tx(bar + 16, 2 * kPanel);
         bulk_copy(p_base + T_ * kPanel, inverse + (chunk_index(t0, seq, ch) * p.heads + h) * (2 * C * C), 2 * kPanel, bar + 16);
       }
@@ -817,7 +819,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
       q_n += __shfl_xor_sync(FULL_MASK, q_n, 1);
 #pragma unroll
       for (int i0 = 0; i0 < 16 * DR; i0 += THREADS) {     // sums of 8 decayed keys, 8 entries of each
-        const int i = i0 + tid, c = i >> 3, tg = i & 7;
+        const int i = i0 + tid, pieces = FULL ? 2 * DR : 2 * k16, tg = i / pieces, c = i - tg * pieces;
         if (i >= 16 * k16) break;
         float acc[8] = {};
 #pragma unroll
