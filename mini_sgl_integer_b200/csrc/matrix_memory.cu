@@ -1049,15 +1049,15 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap map, const MemoryParams 
 // by head: M, the inverses D_i of its four diagonal blocks by substitution, and the blocks below them column by column from
 // T_ij = -D_i sum_(j <= k < i) M_ik T_kj.  The products are transposed as in the chunk kernel, so a block goes from
 // accumulator to left operand in registers; operands are two bf16 numbers each.
-__global__ void __launch_bounds__(128, 4)
+__global__ void __launch_bounds__(128, 5)
 delta_inverse_kernel(const MemoryParams p, const bf16* __restrict__ rows, bf16* __restrict__ inverse) {
   extern __shared__ __align__(128) unsigned char smem[];
   constexpr int C = kChunk;
   const int lk = ((p.dim + 15) & ~15) + 8, k16 = (p.dim + 15) >> 4;
-  unsigned char *mp = smem, *tp = smem + 2 * kPanel;     // M and the inverse: a high and a low panel each
-  float* dg = reinterpret_cast<float*>(tp + 2 * kPanel); // [4][16][16] diagonal blocks of M
+  float* dg = reinterpret_cast<float*>(smem);            // [4][16][16] diagonal blocks of M
   float *ls = dg + 4 * 256, *bs = ls + C, *rk = bs + C, *rq = rk + C;                 // [C] each
-  bf16* ks = reinterpret_cast<bf16*>(rq + C);            // [C][lk]
+  unsigned char *mp = reinterpret_cast<unsigned char*>(rq + C), *tp = mp + 2 * kPanel; // M and the inverse: a high and a low panel each
+  bf16* ks = reinterpret_cast<bf16*>(tp);                // [C][lk] keys, until their products are there
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
@@ -1502,8 +1502,11 @@ static int launch_scan_shape(MemoryParams p, const T* rows, int batch, cudaStrea
 }
 template <int KIND, int DR, bool FULL>
 static int launch_chunk_shape(const CUtensorMap& map, const MemoryParams& p, const bf16* inverse, int batch, cudaStream_t st) {
-  constexpr size_t bytes = chunk_smem(DR, KIND);
-  static_assert(bytes <= 227 * 1024, "shared memory budget");
+  constexpr size_t need = chunk_smem(DR, KIND), alone = 116 * 1024;
+  static_assert(need <= 227 * 1024, "shared memory budget");
+  // few CTAs spread over the SMs (launched while the kernel before still runs, two would share one that is free early)
+  const int64_t ctas = (int64_t)((p.vdim + kChunkCols - 1) / kChunkCols) * p.heads * batch;
+  const size_t bytes = need < alone && ctas <= sm_count() ? alone : need;
   cudaError_t e = cudaFuncSetAttribute(memory_chunk_kernel<KIND, DR, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
   B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
   const dim3 grid((unsigned)((p.vdim + kChunkCols - 1) / kChunkCols), (unsigned)p.heads, (unsigned)batch);
@@ -1523,7 +1526,8 @@ static int launch_chunks(const MemoryParams& p, const bf16* rows, bf16* inverse,
                  B200_E_CUDA, "memory_scan: cuTensorMapEncodeTiled failed");
   }
   if (KIND == B200F_MEMORY_DELTA) {
-    const size_t bytes = (size_t)4 * kPanel + 4 * 256 * 4 + 4 * kChunk * 4 + (size_t)kChunk * (((p.dim + 15) & ~15) + 8) * 2;
+    const size_t keys = (size_t)kChunk * (((p.dim + 15) & ~15) + 8) * 2;
+    const size_t bytes = (size_t)2 * kPanel + 4 * 256 * 4 + 4 * kChunk * 4 + (keys > 2 * kPanel ? keys : 2 * kPanel);
     cudaError_t e = cudaFuncSetAttribute(delta_inverse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
     B200_REQUIRE(e == cudaSuccess, B200_E_CUDA, "memory_scan: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     launch_pdl(delta_inverse_kernel, dim3((unsigned)((max_q + kChunk - 1) / kChunk), (unsigned)p.qk_heads, (unsigned)batch), dim3(128), bytes, st, p, rows, inverse);
