@@ -28,7 +28,8 @@ The script prints ONE JSON line:
 `--impl reference` times only that CPU port (the reference's Python/torch code cannot travel with this
 repository; its arithmetic is restated in oracle/).  Other workloads (`--workload attn|gemm|rowops|prefill|
 tp_layer|tp_linear`) print the same kind of line for one component; `--workload sefevik` prints one for the Sefevik
-design at several sizes, beside the integer model of equal size.
+design at several sizes, beside the integer model of equal size, `--workload derelorn` one for the Derelorn design beside
+Sefevik models of equal size.
 """
 from __future__ import annotations
 

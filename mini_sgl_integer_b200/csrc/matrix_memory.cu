@@ -1348,9 +1348,11 @@ struct MemoryOutput {
   int norm_len;                        // entry i of a row has gain norm_w[i % norm_len]
   float eps;
   int64_t out_pitch;
+  int64_t rows;
+  int wpg, cta_rows;                   // warps per group, rows per CTA
 };
 
-// One CTA per row.  A warp per group, or several for the wide groups of a few; up to kOutKeep packs of a group per lane stay in
+// A CTA per row, or per several short ones.  A warp per group, or several for the wide groups of a few; up to kOutKeep packs of a group per lane stay in
 // registers between the sum of squares and the result, the others are formed twice.
 constexpr int kOutKeep = 2;
 template <int V>
@@ -1362,14 +1364,14 @@ memory_output_kernel(const MemoryOutput p, T* __restrict__ out) {
   __shared__ float part[8];
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t row = blockIdx.x;
   const int n = p.heads * p.vdim, groups = n / p.group;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const float* o = p.o + row * n;
-  const float* gate = p.y + row * p.y_pitch + p.gate_col;
-  const int wpg = groups >= 8 ? 1 : 8 / groups, at_once = 8 / wpg, sub = warp % wpg;       // warps per group
+  const int wpg = p.wpg, at_once = 8 / wpg, sub = warp % wpg;                  // warps per group
+  const int64_t row0 = (int64_t)blockIdx.x * p.cta_rows;
+  const int units = (int)min((int64_t)p.cta_rows, p.rows - row0) * groups;     // (row, group) pairs of this CTA
   const int step = 32 * wpg * V;
   auto load = [&](const float* src) { return *reinterpret_cast<const OutPack<V>*>(src); };
+  const float *o = nullptr, *gate = nullptr;
   auto gate_at = [&](int c) {
     OutPack<V> z = load(gate + c);
     for (int s = 1; s < p.splits; ++s) {
@@ -1379,10 +1381,13 @@ memory_output_kernel(const MemoryOutput p, T* __restrict__ out) {
     }
     return z;
   };
-  for (int g0 = 0; g0 < groups; g0 += at_once) {
-    const int g = g0 + warp / wpg;
-    const bool live = warp / wpg < at_once && g < groups;
-    const int c0 = g * p.group;
+  for (int u0 = 0; u0 < units; u0 += at_once) {
+    const int unit = u0 + warp / wpg;
+    const bool live = warp / wpg < at_once && unit < units;
+    const int r = live ? unit / groups : 0, g = live ? unit - r * groups : 0, c0 = g * p.group;
+    const int64_t row = row0 + r;
+    o = p.o + row * n;
+    gate = p.y + row * p.y_pitch + p.gate_col;
     const float inv_den = live && p.den ? 1.0f / p.den[row * p.heads + g] : 1.0f;         // with den a group is a head
     auto value = [&](int i) {
       OutPack<V> u = load(o + c0 + i);
@@ -1677,11 +1682,15 @@ extern "C" int b200f_memory_output(const float* o, const float* den, int heads, 
                "memory_output: gains of %d for groups of %d, divisors per head of %d", norm_len, group, vdim);
   if (tokens == 0) return B200_OK;
   B200_REQUIRE(o && y && norm_w && out, B200_E_NULL, "memory_output: null pointer");
-  MemoryOutput p{o, den, heads, vdim, group, y, splits, split_stride, y_pitch, gate_col, gate, norm_w, norm_len, eps, out_pitch};
+  MemoryOutput p{o, den, heads, vdim, group, y, splits, split_stride, y_pitch, gate_col, gate, norm_w, norm_len, eps, out_pitch, tokens, 1, 1};
+  const int64_t groups = n / group;
   const bool by4 = group % 4 == 0 && y_pitch % 4 == 0 && gate_col % 4 == 0 && split_stride % 4 == 0 && out_pitch % 4 == 0 && aligned16(o) && aligned16(y) &&
                    aligned16(norm_w) && aligned16(out);
   const int v = by4 && (group >= 128 || group % 2) ? 4 : (by4 && group >= 32 ? 2 : 1);      // narrow packs keep the lanes busy in small groups
-  const dim3 grid((unsigned)tokens), block(256);
+  if (groups < 8 && group > 32 * v * kOutKeep) p.wpg = (int)(8 / groups);
+  else
+    while (p.cta_rows < 8 && (2 * p.cta_rows * n <= 4096 || p.cta_rows * groups < 8) && tokens >= 16ll * p.cta_rows * sm_count()) p.cta_rows *= 2;
+  const dim3 grid((unsigned)((tokens + p.cta_rows - 1) / p.cta_rows)), block(256);
   cudaStream_t st = (cudaStream_t)s;
   if (dtype == B200F_BF16) {
     if (v == 4) launch_pdl(memory_output_kernel<bf16, 4>, grid, block, 0, st, p, (bf16*)out);

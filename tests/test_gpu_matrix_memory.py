@@ -254,6 +254,17 @@ def test_memory_output(dtype, H, V, group):
     close(out, norm(o * S.silu(z)) * w, dtype, 5e-5)
 
 
+@pytest.mark.parametrize("H,V,rows", [(4, 24, 2501), (2, 256, 4801), (1, 100, 2369)])
+def test_memory_output_of_many_short_rows(H, V, rows):
+    """Several rows per CTA, the last one with fewer."""
+    rng = np.random.default_rng(rows)
+    n, eps = H * V, 1e-4
+    o, y, w = rng.standard_normal((rows, n)), rng.standard_normal((1, rows, 2 * n)), rng.standard_normal(n)
+    out = fo.rows(rows, n, torch.bfloat16, "cuda")
+    fo.memory_output(dev(o), None, H, V, V, dev(y), n, fo.GATE_SIGMOID_AFTER, dev(w), eps, out)
+    close(out, S.rms_norm(o.reshape(rows, H, V), 1.0, eps).reshape(rows, n) * w * S.sigmoid(y[0, :, n:]), torch.bfloat16)
+
+
 # ----------------------------------------------------------------------------- gated feed-forward, ends of a sublayer
 @pytest.mark.parametrize("dtype", DT)
 @pytest.mark.parametrize("T,ff,width", [(1, 16, 24), (3, 37, 50), (70, 200, 64), (200, 4096, 128), (300, 130, 72), (1100, 5000, 96), (4, 5000, 2048)])
